@@ -1,5 +1,6 @@
 // Token embedding gather with the additive position table fused in:
-// x[t,:] = table[id_t,:] (+ pos_table[pos_t,:]), written as 32-bit.
+// x[t,:] = table[id_t,:] * scale (+ pos_table[pos_t,:]), written as 32-bit, and once more to `keep` when a later part of the
+// model reads the embedded rows again.
 // Same arithmetic as the reference's embedding_kernel (src/kernels/embedding.cu:23-43),
 // for any width and either table dtype; row offsets are 64-bit.
 #include "common.cuh"
@@ -7,29 +8,31 @@
 template <typename T>
 __global__ void embed_kernel(const int* __restrict__ ids, const int* __restrict__ pos,
                              const T* __restrict__ table, const T* __restrict__ pos_table,
-                             float* __restrict__ out, int D, int copies) {
+                             float* __restrict__ out, float* __restrict__ keep, int D, int copies, float scale) {
     const int t = blockIdx.x;
     pdl_launch();               // the first kernel of a step: nothing before it to wait for
     const T* row = table + (size_t)ids[t] * D;
     const T* prow = pos_table ? pos_table + (size_t)pos[t] * D : nullptr;
     float* o = out + (size_t)t * D * copies;
     for (int d = threadIdx.x; d < D; d += blockDim.x) {
-        float v = to_f32(row[d]);
+        float v = to_f32(row[d]) * scale;
         if (prow) v += to_f32(prow[d]);
+        if (keep) keep[(size_t)t * D + d] = v;
         for (int c = 0; c < copies; ++c) o[(size_t)c * D + d] = v;     // a residual of several streams starts as copies
     }
 }
 
 MLLM_EXPORT int mllm_embed(const int* ids, const int* pos, const void* table, const void* pos_table,
-                           float* out, int T, int D, int copies, int dtype, cudaStream_t stream) {
+                           float* out, float* keep, int T, int D, int copies, float scale, int dtype, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (D <= 0 || copies <= 0) return mllm_fail(1, "embed: width %d, %d copies", D, copies);
     int threads = D >= 256 ? 256 : ((D + 31) / 32) * 32;
     if (dtype == MLLM_F32)
-        embed_kernel<float><<<T, threads, 0, stream>>>(ids, pos, (const float*)table, (const float*)pos_table, out, D, copies);
+        embed_kernel<float><<<T, threads, 0, stream>>>(ids, pos, (const float*)table, (const float*)pos_table, out, keep, D, copies,
+                                                    scale);
     else if (dtype == MLLM_BF16)
         embed_kernel<__nv_bfloat16><<<T, threads, 0, stream>>>(ids, pos, (const __nv_bfloat16*)table,
-                                                               (const __nv_bfloat16*)pos_table, out, D, copies);
+                                                               (const __nv_bfloat16*)pos_table, out, keep, D, copies, scale);
     else
         return mllm_fail(1, "embed: unknown dtype code %d", dtype);
     MLLM_CHECK_LAUNCH("embed");
@@ -53,5 +56,41 @@ MLLM_EXPORT int mllm_resolve_tokens(int* ids, int T, const int* sampled, int row
     if (rows <= 0) return mllm_fail(1, "resolve_tokens: no sampled rows to read from");
     resolve_tokens_kernel<<<(T + 255) / 256, 256, 0, stream>>>(ids, T, sampled, rows);
     MLLM_CHECK_LAUNCH("resolve_tokens");
+    return 0;
+}
+
+// out[t] = [x hi | x0 hi | x lo | x0 lo] (terms = 2, bfloat16: each value as two bfloat16 terms) or [x | x0] (terms = 1):
+// two 32-bit rows side by side as a product reads them.
+template <typename T, int TERMS>
+__global__ void __launch_bounds__(256)
+concat_terms_kernel(const float* x, long long x_stride, const float* x0, long long x0_stride, T* __restrict__ out,
+                    long long out_stride, int D) {
+    pdl_wait();
+    pdl_launch();
+    const size_t t = blockIdx.x;
+    T* o = out + t * out_stride;
+    for (int d = threadIdx.x; d < 2 * D; d += blockDim.x) {
+        const float v = d < D ? x[t * x_stride + d] : x0[t * x0_stride + d - D];
+        const T hi = from_f32<T>(v);
+        o[d] = hi;
+        if (TERMS == 2) o[2 * D + d] = from_f32<T>(v - to_f32(hi));
+    }
+}
+
+MLLM_EXPORT int mllm_concat_terms(const float* x, long long x_stride, const float* x0, long long x0_stride, void* out,
+                                  long long out_stride, int T, int D, int terms, int dtype, cudaStream_t stream) {
+    if (T <= 0) return 0;
+    if (D <= 0) return mllm_fail(1, "concat_terms: width %d", D);
+    if (dtype == MLLM_F32 && terms == 1)
+        MLLM_CUDA(mllm_launch(concat_terms_kernel<float, 1>, dim3(T), dim3(256), 0, stream, true, x, x_stride, x0, x0_stride,
+                              (float*)out, out_stride, D));
+    else if (dtype == MLLM_BF16 && terms == 1)
+        MLLM_CUDA(mllm_launch(concat_terms_kernel<__nv_bfloat16, 1>, dim3(T), dim3(256), 0, stream, true, x, x_stride, x0,
+                              x0_stride, (__nv_bfloat16*)out, out_stride, D));
+    else if (dtype == MLLM_BF16 && terms == 2)
+        MLLM_CUDA(mllm_launch(concat_terms_kernel<__nv_bfloat16, 2>, dim3(T), dim3(256), 0, stream, true, x, x_stride, x0,
+                              x0_stride, (__nv_bfloat16*)out, out_stride, D));
+    else
+        return mllm_fail(1, "concat_terms: %d terms of dtype code %d", terms, dtype);
     return 0;
 }

@@ -5,9 +5,10 @@
 // are small matrix products before and after it.
 //
 //   latent_prepare   per token: RMS norm of the latent (32-bit) -> cache row; rotation of the shared key part and of
-//                    every head's rotated query part at the token's position (angles, cos and sin 32-bit) -> cache row
-//                    and columns R.. of qa.
-//   headwise_linear  out[t][h][n] = sum_k in[t][h][k] W[h][n][k] (optionally times sigmoid(gate[t][h][n])):
+//                    every head's rotated query part at the token's position (angles, cos and sin 32-bit; half-split or
+//                    neighbouring pairs) -> cache row and columns R.. of qa; for queries that go through a latent of their
+//                    own, the RMS norm of that latent too.
+//   headwise_linear  out[t][h][n] = sum_k in[t][h][k] W[h][n][k] (optionally times sigmoid(gate[t][h][n]), or one gate per head):
 //                    the absorbed query (W = W_uk^T per head) and the head outputs (W = W_uv per head, with the gate).
 //                    Three kernels: CUDA-core tiles (32-bit weights, odd sizes), tensor-core tiles (bfloat16 weights,
 //                    more than 16 tokens), and for up to 16 tokens a CTA per (token, head) that streams its weights.
@@ -17,7 +18,9 @@
 //                    sum; online softmax in 32-bit with expf.  Partial (o, m, l) per split, merged in split order by
 //                    latent_merge.  Splits and chunks are fixed ranges of positions, so at one span a token's sums run
 //                    in the same order whether it came in a prompt portion, alone, or in a batch (the caller takes
-//                    short splits for steps of single tokens, to fill the GPU, and long ones otherwise).
+//                    short splits for steps of single tokens, to fill the GPU, and long ones otherwise).  A sink (a
+//                    number per head) adds exp(sink) to the softmax's denominator and to nothing else: the merge starts
+//                    from it, and the tensor-core kernel's running maximum and sum do.
 #include "common.cuh"
 
 namespace {
@@ -31,13 +34,35 @@ template <typename T>
 __global__ void __launch_bounds__(128)
 latent_prepare_kernel(const T* proj, long long ld, int q_off, int dkv_off, int H, int dn, int dr, int R, int rot_dims,
                       const int* positions, const int* slot_mapping, const float* __restrict__ freq, float mscale,
-                      const float* __restrict__ normw, float eps, T* pages, int row, float* qa, int write) {
+                      const float* __restrict__ normw, float eps, T* pages, int row, float* qa, int write, int interleaved,
+                      int dq_off, int q_rank, const float* __restrict__ dq_normw, T* __restrict__ cq, long long ld_cq) {
     __shared__ float scratch[33];
     pdl_wait();
     const int t = blockIdx.x;
     const float p = (float)positions[t];
     const T* x = proj + (size_t)t * ld;
     const int half = rot_dims / 2;
+    // entry i of a rotated part: its pair's frequency, the pair's first and second entry
+    auto turned = [&](const T* v, int i) -> float {
+        const int k = interleaved ? i >> 1 : (i < half ? i : i - half);
+        const int a = interleaved ? 2 * k : k, b = interleaved ? 2 * k + 1 : half + k;
+        float sn, cs;
+        sincosf(p * freq[k], &sn, &cs);
+        sn *= mscale;
+        cs *= mscale;
+        const float u = to_f32(v[a]), w = to_f32(v[b]);
+        return i == a ? u * cs - w * sn : w * cs + u * sn;
+    };
+    if (dq_off >= 0) {                          // the queries' latent, normed for the product that makes queries of it
+        const T* d = x + dq_off;
+        float ss = 0.f;
+        for (int i = threadIdx.x; i < q_rank; i += blockDim.x) {
+            const float v = to_f32(d[i]);
+            ss = fmaf(v, v, ss);
+        }
+        const float r = sqrtf(block_sum(ss, scratch) / (float)q_rank + eps);
+        for (int i = threadIdx.x; i < q_rank; i += blockDim.x) cq[(size_t)t * ld_cq + i] = from_f32<T>(to_f32(d[i]) / r * dq_normw[i]);
+    }
     if (dkv_off >= 0 && write) {
         const T* d = x + dkv_off;
         T* dst = pages + (size_t)slot_mapping[t] * row;
@@ -49,46 +74,29 @@ latent_prepare_kernel(const T* proj, long long ld, int q_off, int dkv_off, int H
         const float r = sqrtf(block_sum(ss, scratch) / (float)R + eps);
         for (int i = threadIdx.x; i < R; i += blockDim.x) dst[i] = from_f32<T>(to_f32(d[i]) / r * normw[i]);
         for (int i = threadIdx.x; i < dr; i += blockDim.x) {
-            float o;
-            if (i < rot_dims) {
-                const int k = i < half ? i : i - half;
-                float sn, cs;
-                sincosf(p * freq[k], &sn, &cs);
-                sn *= mscale;
-                cs *= mscale;
-                const float u = to_f32(d[R + k]), v = to_f32(d[R + half + k]);
-                o = i < half ? u * cs - v * sn : v * cs + u * sn;
-            } else {
-                o = to_f32(d[R + i]);
-            }
-            dst[R + i] = from_f32<T>(o);
+            dst[R + i] = from_f32<T>(i < rot_dims ? turned(d + R, i) : to_f32(d[R + i]));
         }
     }
     const int dq = dn + dr, dk = R + dr;
     for (int j = threadIdx.x; j < H * dr; j += blockDim.x) {
         const int h = j / dr, i = j % dr;
         const T* q = x + q_off + (size_t)h * dq + dn;
-        float o;
-        if (i < rot_dims) {
-            const int k = i < half ? i : i - half;
-            float sn, cs;
-            sincosf(p * freq[k], &sn, &cs);
-            sn *= mscale;
-            cs *= mscale;
-            const float u = to_f32(q[k]), v = to_f32(q[half + k]);
-            o = i < half ? u * cs - v * sn : v * cs + u * sn;
-        } else {
-            o = to_f32(q[i]);
-        }
-        qa[((size_t)t * H + h) * dk + R + i] = o;
+        qa[((size_t)t * H + h) * dk + R + i] = i < rot_dims ? turned(q, i) : to_f32(q[i]);
     }
 }
 
-// out[t][h][n] = sum_k in[t][h][k] * W[h][n][k]  (* sigmoid(gate[t][h * N + n])).  32 tokens x 64 columns per CTA and head.
+// the gate of (t, h, n): gate[t][h * N + n] (gate_n = N), or one per head, gate[t][h] (gate_n = 1)
+template <typename T>
+__device__ __forceinline__ float gate_of(const T* gate, long long ld_gate, int t, int h, int n, int gate_n) {
+    const float z = to_f32(gate[(size_t)t * ld_gate + (gate_n == 1 ? (size_t)h : (size_t)h * gate_n + n)]);
+    return 1.0f / (1.0f + expf(-z));
+}
+
+// out[t][h][n] = sum_k in[t][h][k] * W[h][n][k]  (* sigmoid(the gate)).  32 tokens x 64 columns per CTA and head.
 template <typename TI, typename TW, typename TO>
 __global__ void __launch_bounds__(256)
 headwise_linear_kernel(const TI* in, long long ld_in, int in_head, const TW* __restrict__ W, TO* out, long long ld_out,
-                       int out_head, const TO* gate, long long ld_gate, int Tn, int N, int K) {
+                       int out_head, const TO* gate, long long ld_gate, int gate_n, int Tn, int N, int K) {
     __shared__ float As[32][33];
     __shared__ float Ws[64][33];
     pdl_wait();
@@ -127,7 +135,7 @@ headwise_linear_kernel(const TI* in, long long ld_in, int in_head, const TW* __r
             const int n = n0 + tx + 16 * i;
             if (n >= N) continue;
             float v = acc[j][i];
-            if (gate) v *= 1.0f / (1.0f + expf(-to_f32(gate[(size_t)t * ld_gate + (size_t)h * N + n])));
+            if (gate) v *= gate_of(gate, ld_gate, t, h, n, gate_n);
             out[(size_t)t * ld_out + (size_t)h * out_head + n] = from_f32<TO>(v);
         }
     }
@@ -139,7 +147,7 @@ headwise_linear_kernel(const TI* in, long long ld_in, int in_head, const TW* __r
 template <typename TI, typename TW, typename TO>
 __global__ void __launch_bounds__(256)
 headwise_rows_kernel(const TI* in, long long ld_in, int in_head, const TW* __restrict__ W, TO* out, long long ld_out,
-                     int out_head, const TO* gate, long long ld_gate, int N, int K) {
+                     int out_head, const TO* gate, long long ld_gate, int gate_n, int N, int K) {
     extern __shared__ float hx[];                                // [K]
     pdl_wait();
     const int t = blockIdx.x, h = blockIdx.y;
@@ -163,7 +171,7 @@ headwise_rows_kernel(const TI* in, long long ld_in, int in_head, const TW* __res
         float v = warp_sum(acc[u]);
         const int n = n0 + u;
         if (lane == 0 && n < N) {
-            if (gate) v *= 1.0f / (1.0f + expf(-to_f32(gate[(size_t)t * ld_gate + (size_t)h * N + n])));
+            if (gate) v *= gate_of(gate, ld_gate, t, h, n, gate_n);
             out[(size_t)t * ld_out + (size_t)h * out_head + n] = from_f32<TO>(v);
         }
     }
@@ -297,18 +305,18 @@ latent_attention_kernel(const float* qa, const T* pages, int row, const int* blo
     }
 }
 
-// One warp per (token, head): out = sum_s o_s e^(m_s - M) / sum_s l_s e^(m_s - M) over the splits the token has.
+// One warp per (token, head): out = sum_s o_s e^(m_s - M) / (e^(sink - M) + sum_s l_s e^(m_s - M)) over the token's splits.
 __global__ void __launch_bounds__(256)
 latent_merge_kernel(const float* part_o, const float* part_ml, const int* positions, float* out, int nsplit, int TH, int H,
-                    int R, int span) {
+                    int R, int span, const float* __restrict__ sink) {
     pdl_wait();
     const int th = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (th >= TH) return;
     const int ns = positions[th / H] / span + 1;
     const size_t o = (size_t)th * nsplit;
-    float M = -INFINITY;
+    float M = sink ? sink[th % H] : -INFINITY;
     for (int s = 0; s < ns; ++s) M = fmaxf(M, part_ml[(o + s) * 2]);
-    float L = 0.f;
+    float L = sink ? expf(sink[th % H] - M) : 0.f;
     for (int s = 0; s < ns; ++s) L += part_ml[(o + s) * 2 + 1] * expf(part_ml[(o + s) * 2] - M);
     for (int d = lane; d < R; d += 32) {
         float a = 0.f;
@@ -404,7 +412,7 @@ template <int NO, int CW, int QL>
 __global__ void __launch_bounds__(128 * CW)
 latent_mma_kernel(const float* qa, const __nv_bfloat16* pages, int row, const int* __restrict__ block_table, int bt_stride,
                   const int* __restrict__ tiles, const int* __restrict__ positions, float* out, int H, int R, int dk, int ps,
-                  float scale) {
+                  float scale, const float* __restrict__ sink) {
     using bf = __nv_bfloat16;
     extern __shared__ __align__(16) unsigned char smraw[];
     const int srow = dk + 8;                                     // 16 bytes of padding: ldmatrix rows fall on different banks
@@ -448,6 +456,10 @@ latent_mma_kernel(const float* qa, const __nv_bfloat16* pages, int row, const in
 #pragma unroll
     for (int i = 0; i < NO; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
+    if (sink) {                                                  // in units of ln 2 like the scores; one thread of a row's quad carries its weight
+        m0 = m1 = sink[h] * LOG2E;
+        l0 = l1 = ((lane & 3) == 0 && cs == 0) ? 1.f : 0.f;
+    }
     const int nct = R / 8 - cs * NO;                             // column tiles of 8 this warp has (may exceed NO or be <= 0)
     const int j_last = pos_max / MK;
     for (int j = 0; j <= j_last; ++j) {
@@ -583,7 +595,7 @@ latent_mma_kernel(const float* qa, const __nv_bfloat16* pages, int row, const in
 
 template <int NO, int CW, int QL>
 int launch_mma_q(const float* qa, const void* pages, int row, const int* bt, int bt_stride, const int* tiles, int n_tiles,
-               const int* positions, float* out, int H, int R, int dk, int ps, float scale, cudaStream_t stream) {
+               const int* positions, float* out, int H, int R, int dk, int ps, float scale, const float* sink, cudaStream_t stream) {
     const size_t smem = (size_t)((QL ? 2 : 1) * MQ + 2 * MK) * (dk + 8) * 2 + (CW == 2 ? PAIR_BYTES : 0);
     static bool raised = false;
     if (smem > 48 * 1024 && !raised) {
@@ -591,16 +603,16 @@ int launch_mma_q(const float* qa, const void* pages, int row, const int* bt, int
         raised = true;
     }
     MLLM_CUDA(mllm_launch(latent_mma_kernel<NO, CW, QL>, dim3(H, n_tiles), dim3(128 * CW), smem, stream, true, qa,
-                          (const __nv_bfloat16*)pages, row, bt, bt_stride, tiles, positions, out, H, R, dk, ps, scale));
+                          (const __nv_bfloat16*)pages, row, bt, bt_stride, tiles, positions, out, H, R, dk, ps, scale, sink));
     return 0;
 }
 
 template <int NO, int CW>
 int launch_mma(const float* qa, const void* pages, int row, const int* bt, int bt_stride, const int* tiles, int n_tiles,
-               const int* positions, float* out, int H, int R, int dk, int ps, float scale, cudaStream_t stream) {
+               const int* positions, float* out, int H, int R, int dk, int ps, float scale, const float* sink, cudaStream_t stream) {
     if ((size_t)(2 * MQ + 2 * MK) * (dk + 8) * 2 + (CW == 2 ? PAIR_BYTES : 0) <= MAX_SMEM)
-        return launch_mma_q<NO, CW, 1>(qa, pages, row, bt, bt_stride, tiles, n_tiles, positions, out, H, R, dk, ps, scale, stream);
-    return launch_mma_q<NO, CW, 0>(qa, pages, row, bt, bt_stride, tiles, n_tiles, positions, out, H, R, dk, ps, scale, stream);
+        return launch_mma_q<NO, CW, 1>(qa, pages, row, bt, bt_stride, tiles, n_tiles, positions, out, H, R, dk, ps, scale, sink, stream);
+    return launch_mma_q<NO, CW, 0>(qa, pages, row, bt, bt_stride, tiles, n_tiles, positions, out, H, R, dk, ps, scale, sink, stream);
 }
 
 // The per-head products of many tokens on tensor cores (bfloat16 weights): 64 tokens x 64 columns per CTA and head, K in
@@ -609,7 +621,7 @@ int launch_mma(const float* qa, const void* pages, int row, const int* bt, int b
 template <int MODE>
 __global__ void __launch_bounds__(128)
 headwise_mma_kernel(const void* in_, long long ld_in, int in_head, const __nv_bfloat16* __restrict__ W, void* out_,
-                    long long ld_out, int out_head, const __nv_bfloat16* gate, long long ld_gate, int Tn, int N, int K) {
+                    long long ld_out, int out_head, const __nv_bfloat16* gate, long long ld_gate, int gate_n, int Tn, int N, int K) {
     using bf = __nv_bfloat16;
     constexpr int LD = 72;
     __shared__ __align__(16) bf As[64 * LD];
@@ -672,7 +684,7 @@ headwise_mma_kernel(const void* in_, long long ld_in, int in_head, const __nv_bf
                 if (MODE == 0) {
                     reinterpret_cast<float*>(out_)[(size_t)t * ld_out + (size_t)h * out_head + col] = v;
                 } else {
-                    if (gate) v *= 1.0f / (1.0f + expf(-to_f32(gate[(size_t)t * ld_gate + (size_t)h * N + col])));
+                    if (gate) v *= gate_of(gate, ld_gate, t, h, col, gate_n);
                     reinterpret_cast<bf*>(out_)[(size_t)t * ld_out + (size_t)h * out_head + col] = __float2bfloat16_rn(v);
                 }
             }
@@ -684,31 +696,35 @@ headwise_mma_kernel(const void* in_, long long ld_in, int in_head, const __nv_bf
 
 // proj [T, ...] in `dtype` with row stride ld: queries at column q_off (H heads of dn + dr), the down-projection at
 // dkv_off (R + dr columns; -1: this layer writes no cache row).  pages [slots][row] in `dtype`.  qa [T][H][R + dr] 32-bit:
-// only its columns R.. are written here.
+// only its columns R.. are written here (H = 0: no queries).  dq_off >= 0: columns dq_off .. of q_rank entries are RMS-normed
+// with dq_normw into cq [T][ld_cq].  interleaved: entry 2i of a rotated part pairs with 2i + 1, else i with i + rot_dims / 2.
 MLLM_EXPORT int mllm_latent_prepare(const void* proj, long long ld, int q_off, int dkv_off, int Tn, int H, int dn, int dr,
                                     int R, int rot_dims, const int* positions, const int* slot_mapping, const float* freq,
                                     float mscale, const float* normw, float eps, void* pages, int row, float* qa,
-                                    int write, int dtype, cudaStream_t stream) {
+                                    int write, int interleaved, int dq_off, int q_rank, const float* dq_normw, void* cq,
+                                    long long ld_cq, int dtype, cudaStream_t stream) {
     if (Tn <= 0) return 0;
     if (rot_dims < 0 || rot_dims > dr || rot_dims % 2) return mllm_fail(1, "latent_prepare: %d rotated dimensions of %d", rot_dims, dr);
     if (row < R + dr) return mllm_fail(1, "latent_prepare: cache rows of %d cannot hold %d + %d", row, R, dr);
     if (dtype == MLLM_F32)
         MLLM_CUDA(mllm_launch(latent_prepare_kernel<float>, dim3(Tn), dim3(128), 0, stream, true, (const float*)proj, ld, q_off,
                               dkv_off, H, dn, dr, R, rot_dims, positions, slot_mapping, freq, mscale, normw, eps,
-                              (float*)pages, row, qa, write));
+                              (float*)pages, row, qa, write, interleaved, dq_off, q_rank, dq_normw, (float*)cq, ld_cq));
     else if (dtype == MLLM_BF16)
         MLLM_CUDA(mllm_launch(latent_prepare_kernel<__nv_bfloat16>, dim3(Tn), dim3(128), 0, stream, true,
                               (const __nv_bfloat16*)proj, ld, q_off, dkv_off, H, dn, dr, R, rot_dims, positions, slot_mapping,
-                              freq, mscale, normw, eps, (__nv_bfloat16*)pages, row, qa, write));
+                              freq, mscale, normw, eps, (__nv_bfloat16*)pages, row, qa, write, interleaved, dq_off, q_rank, dq_normw,
+                              (__nv_bfloat16*)cq, ld_cq));
     else
         return mllm_fail(1, "latent_prepare: unknown dtype code %d", dtype);
     return 0;
 }
 
-// mode 0: in `dtype`, W `dtype`, out 32-bit (no gate).  mode 1: in 32-bit, W `dtype`, out `dtype`, optional gate in `dtype`.
+// mode 0: in `dtype`, W `dtype`, out 32-bit (no gate).  mode 1: in 32-bit, W `dtype`, out `dtype`, optional gate in `dtype`
+// (gate_n = N: one per column, 1: one per head).
 MLLM_EXPORT int mllm_headwise_linear(const void* in, long long ld_in, int in_head, const void* W, void* out, long long ld_out,
-                                     int out_head, const void* gate, long long ld_gate, int Tn, int H, int N, int K, int mode,
-                                     int dtype, cudaStream_t stream) {
+                                     int out_head, const void* gate, long long ld_gate, int gate_n, int Tn, int H, int N, int K,
+                                     int mode, int dtype, cudaStream_t stream) {
     if (Tn <= 0 || H <= 0 || N <= 0) return 0;
     if (K <= 0) return mllm_fail(1, "headwise_linear: K = %d", K);
     const dim3 grid((Tn + 31) / 32, (N + 63) / 64, H), block(256);
@@ -719,15 +735,15 @@ MLLM_EXPORT int mllm_headwise_linear(const void* in, long long ld_in, int in_hea
         const size_t smem = (size_t)K * 4;
         if (dtype == MLLM_F32)
             MLLM_CUDA(mllm_launch(headwise_rows_kernel<float, float, float>, rg, block, smem, stream, true, (const float*)in, ld_in,
-                                  in_head, (const float*)W, (float*)out, ld_out, out_head, (const float*)gate, ld_gate, N, K));
+                                  in_head, (const float*)W, (float*)out, ld_out, out_head, (const float*)gate, ld_gate, gate_n, N, K));
         else if (dtype == MLLM_BF16 && mode == 0)
             MLLM_CUDA(mllm_launch(headwise_rows_kernel<__nv_bfloat16, __nv_bfloat16, float>, rg, block, smem, stream, true,
                                   (const __nv_bfloat16*)in, ld_in, in_head, (const __nv_bfloat16*)W, (float*)out, ld_out, out_head,
-                                  (const float*)nullptr, ld_gate, N, K));
+                                  (const float*)nullptr, ld_gate, gate_n, N, K));
         else if (dtype == MLLM_BF16)
             MLLM_CUDA(mllm_launch(headwise_rows_kernel<float, __nv_bfloat16, __nv_bfloat16>, rg, block, smem, stream, true,
                                   (const float*)in, ld_in, in_head, (const __nv_bfloat16*)W, (__nv_bfloat16*)out, ld_out, out_head,
-                                  (const __nv_bfloat16*)gate, ld_gate, N, K));
+                                  (const __nv_bfloat16*)gate, ld_gate, gate_n, N, K));
         else
             return mllm_fail(1, "headwise_linear: unknown dtype code %d", dtype);
         return 0;
@@ -736,27 +752,27 @@ MLLM_EXPORT int mllm_headwise_linear(const void* in, long long ld_in, int in_hea
         const dim3 mg((Tn + 63) / 64, (N + 63) / 64, H);
         if (mode == 0 && ld_in % 8 == 0 && in_head % 8 == 0 && (uintptr_t)in % 16 == 0) {
             MLLM_CUDA(mllm_launch(headwise_mma_kernel<0>, mg, dim3(128), 0, stream, true, in, ld_in, in_head, (const __nv_bfloat16*)W, out,
-                                  ld_out, out_head, (const __nv_bfloat16*)nullptr, ld_gate, Tn, N, K));
+                                  ld_out, out_head, (const __nv_bfloat16*)nullptr, ld_gate, gate_n, Tn, N, K));
             return 0;
         }
         if (mode == 1 && ld_in % 2 == 0 && in_head % 2 == 0 && (uintptr_t)in % 8 == 0) {
             MLLM_CUDA(mllm_launch(headwise_mma_kernel<1>, mg, dim3(128), 0, stream, true, in, ld_in, in_head, (const __nv_bfloat16*)W, out,
-                                  ld_out, out_head, (const __nv_bfloat16*)gate, ld_gate, Tn, N, K));
+                                  ld_out, out_head, (const __nv_bfloat16*)gate, ld_gate, gate_n, Tn, N, K));
             return 0;
         }
     }
     if (dtype == MLLM_F32) {
         MLLM_CUDA(mllm_launch(headwise_linear_kernel<float, float, float>, grid, block, 0, stream, true, (const float*)in, ld_in,
-                              in_head, (const float*)W, (float*)out, ld_out, out_head, (const float*)gate, ld_gate, Tn, N, K));
+                              in_head, (const float*)W, (float*)out, ld_out, out_head, (const float*)gate, ld_gate, gate_n, Tn, N, K));
     } else if (dtype == MLLM_BF16) {
         if (mode == 0)
             MLLM_CUDA(mllm_launch(headwise_linear_kernel<__nv_bfloat16, __nv_bfloat16, float>, grid, block, 0, stream, true,
                                   (const __nv_bfloat16*)in, ld_in, in_head, (const __nv_bfloat16*)W, (float*)out, ld_out,
-                                  out_head, (const float*)nullptr, ld_gate, Tn, N, K));
+                                  out_head, (const float*)nullptr, ld_gate, gate_n, Tn, N, K));
         else
             MLLM_CUDA(mllm_launch(headwise_linear_kernel<float, __nv_bfloat16, __nv_bfloat16>, grid, block, 0, stream, true,
                                   (const float*)in, ld_in, in_head, (const __nv_bfloat16*)W, (__nv_bfloat16*)out, ld_out,
-                                  out_head, (const __nv_bfloat16*)gate, ld_gate, Tn, N, K));
+                                  out_head, (const __nv_bfloat16*)gate, ld_gate, gate_n, Tn, N, K));
     } else {
         return mllm_fail(1, "headwise_linear: unknown dtype code %d", dtype);
     }
@@ -767,8 +783,8 @@ MLLM_EXPORT int mllm_headwise_linear(const void* in, long long ld_in, int in_hea
 // out [T][H][R] 32-bit; part_o [T * H * nsplit * R], part_ml [T * H * nsplit * 2] scratch; nsplit >= ceil(longest context / span).
 MLLM_EXPORT int mllm_latent_attention(const float* qa, const void* pages, int row, const int* block_table, int bt_stride,
                                       const int* token_seq, const int* positions, float* part_o, float* part_ml, int nsplit,
-                                      float* out, int Tn, int H, int R, int dk, int ps, float scale, int span, int dtype,
-                                      cudaStream_t stream) {
+                                      float* out, int Tn, int H, int R, int dk, int ps, float scale, int span, const float* sink,
+                                      int dtype, cudaStream_t stream) {
     if (Tn <= 0) return 0;
     if (R <= 0 || R > MAX_R || dk < R || dk > MAX_DK) return mllm_fail(1, "latent_attention: latent size %d (at most %d), key size %d (at most %d)", R, MAX_R, dk, MAX_DK);
     const int es = dtype == MLLM_F32 ? 4 : 2;
@@ -786,7 +802,7 @@ MLLM_EXPORT int mllm_latent_attention(const float* qa, const void* pages, int ro
         return mllm_fail(1, "latent_attention: unknown dtype code %d", dtype);
     if (rc) return rc;
     MLLM_CUDA(mllm_launch(latent_merge_kernel, dim3((Tn * H + 7) / 8), dim3(256), 0, stream, true, part_o, part_ml, positions,
-                          out, nsplit, Tn * H, H, R, span));
+                          out, nsplit, Tn * H, H, R, span, sink));
     return 0;
 }
 
@@ -799,15 +815,15 @@ MLLM_EXPORT int mllm_latent_mma_ok(int R, int dk, int row) {
 // Prompt portions with a bfloat16 cache: tiles [n_tiles][3] = (request, first flat token, rows <= 64).
 MLLM_EXPORT int mllm_latent_attention_mma(const float* qa, const void* pages, int row, const int* block_table, int bt_stride,
                                           const int* tiles, int n_tiles, const int* positions, float* out, int H, int R,
-                                          int dk, int ps, float scale, cudaStream_t stream) {
+                                          int dk, int ps, float scale, const float* sink, cudaStream_t stream) {
     if (n_tiles <= 0) return 0;
     if (!mllm_latent_mma_ok(R, dk, row) || (uintptr_t)pages % 16 != 0 || (uintptr_t)qa % 8 != 0)
         return mllm_fail(1, "latent_attention_mma: latent %d, key %d, row %d: not sizes this kernel takes", R, dk, row);
     if (n_tiles > 65535) return mllm_fail(1, "latent_attention_mma: too many tiles");
-    if (R <= 32) return launch_mma<4, 1>(qa, pages, row, block_table, bt_stride, tiles, n_tiles, positions, out, H, R, dk, ps, scale, stream);
-    if (R <= 64) return launch_mma<8, 1>(qa, pages, row, block_table, bt_stride, tiles, n_tiles, positions, out, H, R, dk, ps, scale, stream);
-    if (R <= 128) return launch_mma<16, 1>(qa, pages, row, block_table, bt_stride, tiles, n_tiles, positions, out, H, R, dk, ps, scale, stream);
-    if (R <= 256) return launch_mma<16, 2>(qa, pages, row, block_table, bt_stride, tiles, n_tiles, positions, out, H, R, dk, ps, scale, stream);
-    if (R <= 384) return launch_mma<24, 2>(qa, pages, row, block_table, bt_stride, tiles, n_tiles, positions, out, H, R, dk, ps, scale, stream);
-    return launch_mma<32, 2>(qa, pages, row, block_table, bt_stride, tiles, n_tiles, positions, out, H, R, dk, ps, scale, stream);
+    if (R <= 32) return launch_mma<4, 1>(qa, pages, row, block_table, bt_stride, tiles, n_tiles, positions, out, H, R, dk, ps, scale, sink, stream);
+    if (R <= 64) return launch_mma<8, 1>(qa, pages, row, block_table, bt_stride, tiles, n_tiles, positions, out, H, R, dk, ps, scale, sink, stream);
+    if (R <= 128) return launch_mma<16, 1>(qa, pages, row, block_table, bt_stride, tiles, n_tiles, positions, out, H, R, dk, ps, scale, sink, stream);
+    if (R <= 256) return launch_mma<16, 2>(qa, pages, row, block_table, bt_stride, tiles, n_tiles, positions, out, H, R, dk, ps, scale, sink, stream);
+    if (R <= 384) return launch_mma<24, 2>(qa, pages, row, block_table, bt_stride, tiles, n_tiles, positions, out, H, R, dk, ps, scale, sink, stream);
+    return launch_mma<32, 2>(qa, pages, row, block_table, bt_stride, tiles, n_tiles, positions, out, H, R, dk, ps, scale, sink, stream);
 }

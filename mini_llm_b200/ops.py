@@ -41,7 +41,8 @@ def _signatures(lib):
     lib.mllm_set_pdl.argtypes = [c_int]
     lib.mllm_set_pdl.restype = c_int
     sig = {
-        "mllm_embed": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+        "mllm_embed": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p],
+        "mllm_concat_terms": [c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_ll, c_int, c_int, c_int, c_int, c_void_p],
         "mllm_resolve_tokens": [c_void_p, c_int, c_void_p, c_int, c_void_p],
         "mllm_layernorm": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_void_p],
         "mllm_kv_write": [c_void_p, c_void_p, c_ll, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
@@ -127,13 +128,14 @@ def _signatures(lib):
         "mllm_norm_scale_add": [c_void_p, c_ll, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_ll, c_void_p, c_float,
                                 c_float, c_void_p, c_ll, c_int, c_int, c_float, c_int, c_void_p],
         "mllm_latent_prepare": [c_void_p, c_ll, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
-                                c_void_p, c_float, c_void_p, c_float, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p],
+                                c_void_p, c_float, c_void_p, c_float, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int,
+                                c_void_p, c_void_p, c_ll, c_int, c_void_p],
         "mllm_headwise_linear": [c_void_p, c_ll, c_int, c_void_p, c_void_p, c_ll, c_int, c_void_p, c_ll, c_int, c_int, c_int,
-                                 c_int, c_int, c_int, c_void_p],
+                                 c_int, c_int, c_int, c_int, c_void_p],
         "mllm_latent_attention": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
-                                  c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p],
+                                  c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_int, c_void_p],
         "mllm_latent_attention_mma": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int,
-                                      c_int, c_int, c_int, c_float, c_void_p],
+                                      c_int, c_int, c_int, c_float, c_void_p, c_void_p],
         "mllm_latent_mma_ok": [c_int, c_int, c_int],
         "mllm_ssd_conv": [c_void_p, c_ll, c_int, c_void_p, c_void_p, c_void_p, c_ll, c_int, c_void_p, c_void_p, c_void_p,
                           c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
@@ -141,6 +143,20 @@ def _signatures(lib):
                           c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
         "mllm_gated_group_norm": [c_void_p, c_void_p, c_ll, c_void_p, c_void_p, c_ll, c_int, c_int, c_int, c_float, c_int,
                                   c_void_p],
+        "mllm_attention_mixed_chunk": [],
+        "mllm_attention_mixed_ok": [c_int, c_int, c_int, c_int],
+        "mllm_attention_mixed_mma_ok": [c_int, c_int, c_int, c_int],
+        "mllm_attention_mixed": [c_void_p, c_ll, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
+                                 c_ll, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p,
+                                 c_int, c_void_p, c_int, c_int, c_void_p],
+        "mllm_mlstm_max_dim": [],
+        "mllm_mlstm_step_ok": [c_int, c_int],
+        "mllm_mlstm_scan": [c_void_p, c_ll, c_int, c_int, c_int, c_int, c_int, c_void_p, c_ll, c_void_p, c_void_p, c_void_p, c_void_p,
+                            c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p],
+        "mllm_mlstm_finish": [c_void_p, c_void_p, c_void_p, c_ll, c_int, c_void_p, c_void_p, c_ll, c_void_p, c_void_p, c_void_p,
+                              c_void_p, c_ll, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_int, c_int, c_void_p],
+        "mllm_mlstm_step": [c_void_p, c_ll, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_ll, c_void_p, c_void_p, c_void_p,
+                            c_void_p, c_ll, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_float, c_int, c_int, c_void_p],
         "mllm_moe_route": [c_void_p, c_ll, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
                            c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
         "mllm_moe_grouped": [c_void_p, c_ll, c_void_p, c_void_p, c_ll, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
@@ -338,9 +354,10 @@ def _rows(name: str, t: torch.Tensor):
 
 
 # --------------------------------------------------------------------------- embedding
-def embed(ids, positions, table, pos_table, out, copies: int = 1) -> None:
-    """out[t] = table[ids[t]] (+ pos_table[positions[t]]), 32-bit; with ``copies`` > 1 a row of out holds that many
-    copies of the token's row side by side (a residual of several streams at its start)."""
+def embed(ids, positions, table, pos_table, out, copies: int = 1, scale: float = 1.0, keep=None) -> None:
+    """out[t] = table[ids[t]] * scale (+ pos_table[positions[t]]), 32-bit; with ``copies`` > 1 a row of out holds that many
+    copies of the token's row side by side (a residual of several streams at its start).  ``keep`` (32-bit [T, D]): the
+    row once more, for a part that reads it later in the step."""
     _cuda("ids", ids, torch.int32)
     _cuda("table", table)
     _cuda("out", out, torch.float32)
@@ -350,6 +367,10 @@ def embed(ids, positions, table, pos_table, out, copies: int = 1) -> None:
     D //= copies
     if ids.numel() != T or table.shape[1] != D:
         raise KernelError(f"embed: {ids.numel()} ids, table {tuple(table.shape)}, out {tuple(out.shape)}")
+    if keep is not None:
+        _cuda("keep", keep, torch.float32)
+        if tuple(keep.shape) != (T, D):
+            raise KernelError(f"embed: keep {tuple(keep.shape)} for {T} rows of {D}")
     pp = None
     if pos_table is not None:
         _cuda("positions", positions, torch.int32)
@@ -358,7 +379,22 @@ def embed(ids, positions, table, pos_table, out, copies: int = 1) -> None:
             raise KernelError("embed: position table or positions do not fit")
         pp = pos_table.data_ptr()
     _call("mllm_embed", ids.data_ptr(), positions.data_ptr() if pos_table is not None else None,
-          table.data_ptr(), pp, out.data_ptr(), T, D, int(copies), _dt(table), _stream())
+          table.data_ptr(), pp, out.data_ptr(), keep.data_ptr() if keep is not None else None, T, D, int(copies), float(scale),
+          _dt(table), _stream())
+
+
+def concat_terms(x, x0, out, terms: int) -> None:
+    """out[t] = [x[t] | x0[t]] for a product that reads both (``terms`` 1), or [x hi | x0 hi | x lo | x0 lo] with every
+    32-bit value as two bfloat16 terms, the second the rest of the first (``terms`` 2)."""
+    _cuda("x", x, torch.float32, contiguous=False)
+    _cuda("x0", x0, torch.float32, contiguous=False)
+    _cuda("out", out, contiguous=False)
+    T, D = x.shape
+    if tuple(x0.shape) != (T, D) or tuple(out.shape) != (T, 2 * D * terms) or terms not in (1, 2) \
+            or (terms == 2 and out.dtype != torch.bfloat16):
+        raise KernelError(f"concat_terms: x {tuple(x.shape)}, x0 {tuple(x0.shape)}, out {tuple(out.shape)} {out.dtype}, {terms} terms")
+    _call("mllm_concat_terms", x.data_ptr(), _rows("x", x), x0.data_ptr(), _rows("x0", x0), out.data_ptr(), _rows("out", out), T, D,
+          int(terms), _dt(out), _stream())
 
 
 def resolve_tokens(ids, sampled) -> None:
@@ -902,6 +938,83 @@ def biased_attention(q, k_pages, v_pages, block_table, ctx, out, *, num_heads, n
 
 
 
+# --------------------------------------------------------------------------- attention with scores mixed over the heads
+MIXED_ATTN_MAX_DIM, MIXED_ATTN_MAX_HEADS = 256, 64       # what csrc/attention_mixed.cu takes
+
+
+def mixed_attention_ok(heads: int, kv_heads: int, dk: int, dv: int) -> bool:
+    """Whether the kernels take these sizes (dk: a key row of the pages)."""
+    return library().mllm_attention_mixed_ok(heads, kv_heads, dk, dv) == 1
+
+
+def mixed_attention(q, k_pages, v_pages, block_table, ctx, out, *, num_heads, num_kv_heads, scale, mix, window=None, sink=None,
+                    impl: Optional[str] = None) -> None:
+    """Causal attention over the cache whose scores are mixed over the heads before the softmax: with r_g = (q_g . k) * scale
+    the raw scores of the heads, s_h = sum_g mix[h, g] r_g (``mix`` float32 [heads, heads]); softmax over the visible keys
+    (the last ``window``, or all) with exp(sink[h]) added to the denominator (``sink`` float32 [heads], or None); the weighted
+    sum of head h's own values.  q [T, heads * dkq], k_pages [P, kv_heads, page_size, dk] with dk >= dkq a multiple of 8 (rows
+    padded with zeros), v_pages [P, kv_heads, page_size, dv], out [T, heads * dv].
+
+    ``impl``: "split" (single tokens), "rows" (prompt portions, CUDA cores), "mma" (prompt portions, bfloat16, tensor cores);
+    None picks by the step's shape."""
+    _cuda("q", q, contiguous=False)
+    _cuda("k_pages", k_pages, q.dtype)
+    _cuda("v_pages", v_pages, q.dtype)
+    _cuda("out", out, q.dtype, contiguous=False)
+    _cuda("block_table", block_table, torch.int32, contiguous=False)
+    _cuda("mix", mix, torch.float32)
+    T = q.shape[0]
+    _, G, ps, dk = k_pages.shape
+    dv = v_pages.shape[3]
+    dkq = q.shape[1] // num_heads
+    if G != num_kv_heads or q.shape[1] != num_heads * dkq or not (0 < dkq <= dk) or tuple(out.shape) != (T, num_heads * dv) \
+            or v_pages.shape[:3] != k_pages.shape[:3] or tuple(mix.shape) != (num_heads, num_heads):
+        raise KernelError("mixed_attention: head counts or sizes do not fit the pages")
+    if not mixed_attention_ok(num_heads, G, dk, dv):
+        raise KernelError(f"mixed_attention: {num_heads} heads over {G} of sizes {dk} / {dv}")
+    if sink is not None:
+        _cuda("sink", sink, torch.float32)
+        if sink.numel() != num_heads:
+            raise KernelError("mixed_attention: one sink per query head")
+    ldq, ldo = _rows("q", q), _rows("out", out)
+    mma_ok = (q.dtype == torch.bfloat16 and dkq == dk and ldq % 8 == 0 and q.data_ptr() % 16 == 0 and ldo % 2 == 0
+              and out.data_ptr() % 4 == 0 and v_pages.data_ptr() % 16 == 0
+              and library().mllm_attention_mixed_mma_ok(num_heads, G, dk, dv) == 1)
+    tiled = getattr(ctx, "n_tiles", 0) > 0
+    if impl is None:
+        impl = "split" if getattr(ctx, "decode_only", False) or not tiled else ("mma" if mma_ok else "rows")
+    if impl not in ("split", "rows", "mma"):
+        raise KernelError(f"mixed_attention: unknown implementation {impl!r}")
+    if impl == "mma" and not mma_ok:
+        raise KernelError("mixed_attention: the tensor-core kernel takes bfloat16, up to 32 heads, key sizes that are multiples of "
+                          "16 and value sizes of 8 up to 128, and 16-byte aligned rows")
+    if impl != "split" and not tiled:
+        raise KernelError("mixed_attention: prompt portions need the step's tile list")
+    attention_launches["mixed_" + impl] = attention_launches.get("mixed_" + impl, 0) + 1
+    part_o = part_ml = None
+    nsplit = 0
+    if impl == "split":
+        nsplit = mixed_splits(ctx.max_ctx_len, window)
+        part_o = ctx.ws.buf("mattn_part_o", T * num_heads * nsplit, dv, torch.float32).data_ptr()
+        part_ml = ctx.ws.buf("mattn_part_ml", T * num_heads * nsplit, 2, torch.float32).data_ptr()
+    _call("mllm_attention_mixed", q.data_ptr(), ldq, k_pages.data_ptr(), v_pages.data_ptr(), block_table.data_ptr(),
+          _rows("block_table", block_table), ctx.token_seq.data_ptr(), ctx.positions.data_ptr(),
+          ctx.attn_tiles.data_ptr() if impl != "split" else None, int(ctx.n_tiles) if impl != "split" else 0, out.data_ptr(), ldo,
+          part_o, part_ml, nsplit, T, num_heads, G, dkq, dk, dv, ps, float(scale), mix.data_ptr(), int(window or 0),
+          sink.data_ptr() if sink is not None else None, _dt(q), {"rows": 0, "split": 1, "mma": 2}[impl], _stream())
+    if impl == "split":
+        global launches
+        launches += 1           # the kernel that merges the chunks
+
+
+def mixed_splits(max_ctx_len: int, window=None) -> int:
+    """Chunks of keys that a single token sees at most: as many as the context has (rounded so that the number follows from
+    ``latent_splits``, which is part of a step's shape for captured graphs), or the window can touch."""
+    chunk = int(library().mllm_attention_mixed_chunk())
+    n = max(1, latent_splits(max_ctx_len) * LATENT_SPAN_DECODE // chunk)
+    return n if not window else min(n, (int(window) + chunk - 2) // chunk + 1)
+
+
 # --------------------------------------------------------------------------- normed and rotated queries and keys
 def qk_norm_rope(proj, q_off: int, k_off: int, v_off: int, ctx, q_out, k_pages, v_pages, slot_mapping, *, heads: int,
                  kv_heads: int, head_dim: int, v_head_dim: int, q_norm=None, k_norm=None, eps: float = 0.0, freq=None,
@@ -1228,15 +1341,24 @@ LATENT_SPAN_DECODE, LATENT_SPAN_PROMPT = 128, 1024
 
 
 def latent_prepare(proj, q_off: int, dkv_off: Optional[int], ctx, slot_mapping, freq, mscale: float, norm_weight, eps: float,
-                   pages, qa, *, heads: int, dim: int, rot_dim: int, rank: int, rot_dims: int, write: bool) -> None:
+                   pages, qa, *, heads: int, dim: int, rot_dim: int, rank: int, rot_dims: int, write: bool,
+                   interleaved: bool = False, dq_norm=None, cq=None) -> None:
     """Per token of the step: the latent (columns dkv_off .. of ``proj``, RMS-normed with ``norm_weight``) and the shared
     key part rotated at the token's position go to the token's cache row [rank | rot_dim | padding] (``dkv_off`` None or
     ``write`` False: no row is written); every head's rotated query part goes, rotated, to columns rank.. of
-    qa [T, heads, rank + rot_dim] (32-bit).  Angles p * freq[i], cos and sin times ``mscale``, all 32-bit."""
+    qa [T, heads, rank + rot_dim] (32-bit).  Angles p * freq[i], cos and sin times ``mscale``, all 32-bit.  ``interleaved``:
+    entry 2i of a rotated part pairs with 2i + 1, else i with i + rot_dims / 2.  ``heads`` 0 (qa None): no queries.
+    ``dq_norm`` (float32) and ``cq``: the columns q_off .. are not queries but their latent, RMS-normed into cq."""
     _cuda("proj", proj, contiguous=False)
-    _cuda("qa", qa, torch.float32)
+    if heads:
+        _cuda("qa", qa, torch.float32)
     _cuda("freq", freq, torch.float32)
     T = proj.shape[0]
+    if dq_norm is not None:
+        _cuda("dq_norm", dq_norm, torch.float32)
+        _cuda("cq", cq, proj.dtype, contiguous=False)
+        if heads or tuple(cq.shape) != (T, dq_norm.numel()) or q_off + dq_norm.numel() > proj.shape[1]:
+            raise KernelError(f"latent_prepare: the queries' latent {tuple(cq.shape)} against {dq_norm.numel()} weights")
     row = 0
     if dkv_off is not None and write:
         _cuda("pages", pages, proj.dtype)
@@ -1247,24 +1369,27 @@ def latent_prepare(proj, q_off: int, dkv_off: Optional[int], ctx, slot_mapping, 
             raise KernelError("latent_prepare: the cache must have one key/value head and one slot per token")
     else:
         row = rank + rot_dim
-    if tuple(qa.shape) != (T, heads * (rank + rot_dim)) or freq.numel() * 2 != rot_dims:
-        raise KernelError(f"latent_prepare: qa {tuple(qa.shape)} for {heads} heads of {rank} + {rot_dim}")
+    if (heads and tuple(qa.shape) != (T, heads * (rank + rot_dim))) or freq.numel() * 2 != rot_dims:
+        raise KernelError(f"latent_prepare: {heads} heads of {rank} + {rot_dim}, {freq.numel()} frequencies")
     wr = dkv_off is not None and write
     _call("mllm_latent_prepare", proj.data_ptr(), _rows("proj", proj), int(q_off), int(dkv_off) if wr else -1, T, heads, dim,
           rot_dim, rank, rot_dims, ctx.positions.data_ptr(), slot_mapping.data_ptr() if wr else None, freq.data_ptr(),
           float(mscale), norm_weight.data_ptr() if wr else None, float(eps), pages.data_ptr() if wr else None, row,
-          qa.data_ptr(), int(wr), _dt(proj), _stream())
+          qa.data_ptr() if heads else None, int(wr), int(bool(interleaved)), int(q_off) if dq_norm is not None else -1,
+          dq_norm.numel() if dq_norm is not None else 0, dq_norm.data_ptr() if dq_norm is not None else None,
+          cq.data_ptr() if dq_norm is not None else None, _rows("cq", cq) if dq_norm is not None else 0, _dt(proj), _stream())
 
 
 def headwise_linear(x, x_head: int, weight, out, out_head: int, gate=None) -> None:
-    """out[t, h*out_head + n] = sum_k x[t, h*x_head + k] * weight[h, n, k], optionally times sigmoid(gate[t, h*N + n]):
-    a small product per head.  Either x has the weights' dtype and out is 32-bit, or x is 32-bit and out (and the
+    """out[t, h*out_head + n] = sum_k x[t, h*x_head + k] * weight[h, n, k], optionally times sigmoid(gate[t, h*N + n]) or,
+    with a gate of one column per head, sigmoid(gate[t, h]): a small product per head.  Either x has the weights' dtype and out is 32-bit, or x is 32-bit and out (and the
     gate) have the weights' dtype."""
     _cuda("x", x, contiguous=False)
     _cuda("weight", weight)
     _cuda("out", out, contiguous=False)
     H, N, K = weight.shape
     T = x.shape[0]
+    gate_n = N
     if out.shape[0] != T or x_head < K or out_head < N:
         raise KernelError("headwise_linear: shapes do not fit the weights")
     if x.dtype == weight.dtype and out.dtype == torch.float32 and gate is None:
@@ -1273,18 +1398,22 @@ def headwise_linear(x, x_head: int, weight, out, out_head: int, gate=None) -> No
         mode = 1
         if gate is not None:
             _cuda("gate", gate, weight.dtype, contiguous=False)
+            if gate.shape[0] != T or gate.shape[1] not in (H, H * N):
+                raise KernelError(f"headwise_linear: gate {tuple(gate.shape)} for {H} heads of {N}")
+            gate_n = N if gate.shape[1] == H * N else 1
     else:
         raise KernelError(f"headwise_linear: x {x.dtype}, weight {weight.dtype}, out {out.dtype}")
     _call("mllm_headwise_linear", x.data_ptr(), _rows("x", x), int(x_head), weight.data_ptr(), out.data_ptr(), _rows("out", out),
           int(out_head), gate.data_ptr() if gate is not None else None, _rows("gate", gate) if gate is not None else 0,
-          T, H, N, K, mode, _dt(weight), _stream())
+          gate_n, T, H, N, K, mode, _dt(weight), _stream())
 
 
-def latent_attention(qa, pages, block_table, ctx, out, *, heads: int, rank: int, scale: float,
+def latent_attention(qa, pages, block_table, ctx, out, *, heads: int, rank: int, scale: float, sink=None,
                      impl: Optional[str] = None) -> None:
     """Causal softmax attention of qa [T, heads * dk] (32-bit) over cache rows pages [P, 1, page_size, row]: a token's row
     holds its key (the first dk columns) and its value (the first ``rank`` columns) for all heads.
-    out[t, h] = sum_j softmax_j((qa[t, h] . row_j[:dk]) * scale) row_j[:rank], 32-bit [T, heads * rank].
+    out[t, h] = sum_j softmax_j((qa[t, h] . row_j[:dk]) * scale) row_j[:rank], 32-bit [T, heads * rank].  ``sink`` (float32
+    [heads]): exp(sink[h]) is one more term of the softmax's denominator and of nothing else.
     ``impl``: "split" (CUDA cores, all 32-bit, splits of 256 keys: single tokens, 32-bit caches, any size) or "mma"
     (tensor cores: steps with prompt portions over a bfloat16 cache); None picks by the step's shape."""
     _cuda("qa", qa, torch.float32)
@@ -1298,6 +1427,12 @@ def latent_attention(qa, pages, block_table, ctx, out, *, heads: int, rank: int,
         raise KernelError("latent_attention: shapes do not fit the cache rows")
     if rank > LATENT_MAX_RANK or dk > LATENT_MAX_KEY:
         raise KernelError(f"latent_attention: latent size {rank} (at most {LATENT_MAX_RANK}), key size {dk} (at most {LATENT_MAX_KEY})")
+    sink_ptr = None
+    if sink is not None:
+        _cuda("sink", sink, torch.float32)
+        if sink.numel() != heads:
+            raise KernelError(f"latent_attention: {sink.numel()} sinks for {heads} heads")
+        sink_ptr = sink.data_ptr()
     mma_ok = pages.dtype == torch.bfloat16 and getattr(ctx, "n_tiles", 0) > 0 and library().mllm_latent_mma_ok(rank, dk, row) == 1
     if impl is None:
         impl = "mma" if mma_ok and not getattr(ctx, "decode_only", False) else "split"
@@ -1308,7 +1443,7 @@ def latent_attention(qa, pages, block_table, ctx, out, *, heads: int, rank: int,
                               "that are multiples of 8 and keys that are multiples of 16")
         _call("mllm_latent_attention_mma", qa.data_ptr(), pages.data_ptr(), row, block_table.data_ptr(),
               _rows("block_table", block_table), ctx.attn_tiles.data_ptr(), int(ctx.n_tiles), ctx.positions.data_ptr(),
-              out.data_ptr(), heads, rank, dk, ps, float(scale), _stream())
+              out.data_ptr(), heads, rank, dk, ps, float(scale), sink_ptr, _stream())
         return
     if impl != "split":
         raise KernelError(f"latent_attention: unknown implementation {impl!r}")
@@ -1319,7 +1454,7 @@ def latent_attention(qa, pages, block_table, ctx, out, *, heads: int, rank: int,
     part_ml = ctx.ws.buf("latent_part_ml", T * heads * nsplit, 2, torch.float32)
     _call("mllm_latent_attention", qa.data_ptr(), pages.data_ptr(), row, block_table.data_ptr(), _rows("block_table", block_table),
           ctx.token_seq.data_ptr(), ctx.positions.data_ptr(), part_o.data_ptr(), part_ml.data_ptr(), nsplit, out.data_ptr(),
-          T, heads, rank, dk, ps, float(scale), span, _dt(pages), _stream())
+          T, heads, rank, dk, ps, float(scale), span, sink_ptr, _dt(pages), _stream())
     global launches
     launches += 1           # the kernel that merges the splits
 
@@ -1328,6 +1463,76 @@ def latent_splits(max_ctx_len: int) -> int:
     """Splits of the latent attention at a context length (part of a step's shape for captured graphs)."""
     need = max(1, -(-int(max_ctx_len) // LATENT_SPAN_DECODE))
     return 1 << (need - 1).bit_length()
+
+
+# --------------------------------------------------------------------------- matrix memory
+MLSTM_MAX_DIM = 256      # most rows and columns of a head's state that csrc/mlstm.cu takes
+
+
+def _mlstm_sizes(name: str, proj, cols: dict, state, heads: int, dim: int, vdim: int) -> None:
+    _cuda("proj", proj, torch.float32, contiguous=False)
+    _cuda("state", state, torch.float32)
+    width = {"q": heads * dim, "k": heads * dim, "v": heads * vdim, "g": heads * vdim, "i": heads, "f": heads}
+    for c, at in cols.items():
+        if at < 0 or at + width[c] > proj.shape[1]:
+            raise KernelError(f"{name}: columns of {c!r} at {at} in rows of {proj.shape[1]}")
+    if state.dim() != 2 or state.shape[1] < heads * (dim * (vdim + 1) + 1):
+        raise KernelError(f"{name}: a state row of {state.shape[-1]} floats for {heads} heads of {dim} x {vdim}")
+
+
+def mlstm_scan(proj, cols: dict, state, ctx, raw, aux, *, heads: int, dim: int, vdim: int, cap: float, write_state: bool = True,
+               want_cols: int = 0) -> None:
+    """The recurrence of a matrix memory with exponential gates over the step's tokens, request by request and head by head.
+    proj 32-bit [T, .] with the columns ``cols`` = {"q", "k", "v", "i", "f"} -> first column; i = cap * tanh(./cap),
+    f = logsigmoid(cap * tanh(./cap)), m' = max(f + m, i), S <- exp(f + m - m') S + exp(i - m') k v^T, n likewise with k alone.
+    state [slots, >= heads * (dim * (vdim + 1) + 1)]: S [heads, dim, vdim], n [heads, dim], m [heads] (m is written by
+    ``mlstm_finish``).  raw [T, heads * vdim] = S^T q, aux [T, heads * 2] = (n . q, m)."""
+    _mlstm_sizes("mlstm_scan", proj, {c: cols[c] for c in "qkvif"}, state, heads, dim, vdim)
+    _cuda("raw", raw, torch.float32)
+    _cuda("aux", aux, torch.float32)
+    T = proj.shape[0]
+    if tuple(raw.shape) != (T, heads * vdim) or tuple(aux.shape) != (T, heads * 2):
+        raise KernelError("mlstm_scan: raw or aux does not fit")
+    _call("mllm_mlstm_scan", proj.data_ptr(), _rows("proj", proj), cols["q"], cols["k"], cols["v"], cols["i"], cols["f"],
+          state.data_ptr(), state.stride(0), ctx.cu_q.data_ptr(), ctx.state_slots.data_ptr(), raw.data_ptr(), aux.data_ptr(), ctx.S,
+          heads, dim, vdim, float(cap), int(write_state), int(want_cols), _stream())
+
+
+def mlstm_finish(raw, aux, proj, cols: dict, weight, state, ctx, out, *, heads: int, dim: int, vdim: int, q_scale: float,
+                 denom_eps: float, eps: float, write_state: bool = True) -> None:
+    """out = u(o) * weight * sigmoid(g) per head, with o = q_scale raw / (max(|q_scale n.q|, exp(-m)) + denom_eps), u(o) = o
+    over its root mean square (eps inside the root), g the columns ``cols["g"]`` of proj; every request's last m goes to its
+    state."""
+    _mlstm_sizes("mlstm_finish", proj, {"g": cols["g"]}, state, heads, dim, vdim)
+    _cuda("weight", weight, torch.float32)
+    _cuda("out", out, contiguous=False)
+    T = proj.shape[0]
+    if tuple(out.shape) != (T, heads * vdim) or weight.numel() != heads * vdim or tuple(raw.shape) != (T, heads * vdim):
+        raise KernelError("mlstm_finish: shapes do not fit")
+    _call("mllm_mlstm_finish", raw.data_ptr(), aux.data_ptr(), proj.data_ptr(), _rows("proj", proj), cols["g"], weight.data_ptr(),
+          state.data_ptr(), state.stride(0), ctx.token_seq.data_ptr(), ctx.cu_q.data_ptr(), ctx.state_slots.data_ptr(),
+          out.data_ptr(), _rows("out", out), T, heads, dim, vdim, float(q_scale), float(denom_eps), float(eps), int(write_state),
+          _dt(out), _stream())
+
+
+def mlstm_step_ok(dim: int, vdim: int) -> bool:
+    """Whether the single-launch kernel takes steps of single tokens of these sizes."""
+    return library().mllm_mlstm_step_ok(dim, vdim) == 1
+
+
+def mlstm_step(proj, cols: dict, weight, state, ctx, out, *, heads: int, dim: int, vdim: int, cap: float, q_scale: float,
+               denom_eps: float, eps: float, write_state: bool = True) -> None:
+    """``mlstm_scan`` and ``mlstm_finish`` of a step of single tokens in one launch (the same state bit for bit)."""
+    _mlstm_sizes("mlstm_step", proj, cols, state, heads, dim, vdim)
+    _cuda("weight", weight, torch.float32)
+    _cuda("out", out, contiguous=False)
+    T = proj.shape[0]
+    if tuple(out.shape) != (T, heads * vdim) or weight.numel() != heads * vdim:
+        raise KernelError("mlstm_step: shapes do not fit")
+    _call("mllm_mlstm_step", proj.data_ptr(), _rows("proj", proj), cols["q"], cols["k"], cols["v"], cols["g"], cols["i"], cols["f"],
+          state.data_ptr(), state.stride(0), ctx.cu_q.data_ptr(), ctx.state_slots.data_ptr(), weight.data_ptr(), out.data_ptr(),
+          _rows("out", out), ctx.S, heads, dim, vdim, float(cap), float(q_scale), float(denom_eps), float(eps), int(write_state),
+          _dt(out), _stream())
 
 
 # --------------------------------------------------------------------------- state-space mixer

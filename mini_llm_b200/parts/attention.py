@@ -320,3 +320,96 @@ class RotaryAttention(ProjectedMixer):
 
 
 register_part("mixer", "rotary_attention", RotaryAttention)
+
+
+class MixedScoreAttention(ProjectedMixer):
+    """Causal softmax attention with grouped key/value heads, key and value heads of different sizes, no positions, and scores
+    that are mixed over the query heads before the softmax: s_h = sum_g talk[h, g] * (q_g . k) * scale, ``talk`` a learned
+    [heads, heads] matrix (query head g reads key/value head floor(g / (heads / kv_heads))).
+
+    Options, all constructor constants.  ``window``: a query sees itself and the window - 1 tokens before it.  ``bias``: the
+    three input projections have biases; ``out_bias``: so has the output projection.  ``sink``: "zero" (one is added to the
+    softmax's denominator: a sink whose score is 0), "learned" (exp of a trained scalar per head is) or None.
+
+    Every head needs the raw scores of all the others, so a CTA of the kernels takes all heads of its queries."""
+
+    in_names = ("q_weight", "k_weight", "v_weight")
+    out_name = "out_weight"
+
+    def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, head_dim: int, v_head_dim: int, scale: float,
+                 window: Optional[int] = None, bias: bool = False, out_bias: bool = False, sink: Optional[str] = None):
+        self.hidden_size, self.num_heads, self.num_kv_heads = int(hidden_size), int(num_heads), int(num_kv_heads)
+        self.head_dim, self.v_head_dim = int(head_dim), int(v_head_dim)
+        self.scale = float(scale)
+        self.window = None if window is None else int(window)
+        self.has_bias, self.has_out_bias = bool(bias), bool(out_bias)
+        if sink not in (None, "zero", "learned"):
+            raise ValueError(f"mixed-score attention: sink is None, 'zero' or 'learned', got {sink!r}")
+        self.sink_kind = sink
+        if self.num_heads % self.num_kv_heads != 0:
+            raise ValueError(f"num_heads={num_heads} is not a multiple of num_kv_heads={num_kv_heads}")
+        if self.window is not None and self.window < 1:
+            raise ValueError("the window must be positive")
+        self.q_size = self.num_heads * self.head_dim
+        self.k_size = self.num_kv_heads * self.head_dim
+        self.v_size = self.num_kv_heads * self.v_head_dim
+        self.k_row = -(-self.head_dim // 8) * 8        # a key row in the pages: padded to 16-byte pieces, the padding zero
+        self.sink = None
+
+    def param_specs(self):
+        H = self.num_heads
+        p = {"q_weight": ParamSpec((self.q_size, self.hidden_size), "matrix"),
+             "k_weight": ParamSpec((self.k_size, self.hidden_size), "matrix"),
+             "v_weight": ParamSpec((self.v_size, self.hidden_size), "matrix"),
+             "talk": ParamSpec((H, H), "vector"),       # 32-bit: it acts on scores
+             "out_weight": ParamSpec((self.hidden_size, H * self.v_head_dim), "matrix")}
+        if self.has_bias:
+            p["q_bias"] = ParamSpec((self.q_size,), "vector")
+            p["k_bias"] = ParamSpec((self.k_size,), "vector")
+            p["v_bias"] = ParamSpec((self.v_size,), "vector")
+        if self.has_out_bias:
+            p["out_bias"] = ParamSpec((self.hidden_size,), "vector")
+        if self.sink_kind == "learned":
+            p["sink"] = ParamSpec((H,), "vector")
+        return p
+
+    def kernel_limits(self, dtype: str):
+        from .. import ops
+        out = []
+        if self.num_heads > ops.MIXED_ATTN_MAX_HEADS:
+            out.append(f"mixed-score attention: {self.num_heads} heads; the kernels take {ops.MIXED_ATTN_MAX_HEADS}")
+        if max(self.head_dim, self.v_head_dim) > ops.MIXED_ATTN_MAX_DIM:
+            out.append(f"mixed-score attention: keys of {self.head_dim} and values of {self.v_head_dim}; the kernels take up to "
+                       f"{ops.MIXED_ATTN_MAX_DIM}")
+        if not out and not ops.mixed_attention_ok(self.num_heads, self.num_kv_heads, self.k_row, self.v_head_dim):
+            out.append(f"mixed-score attention: {self.num_heads} heads of {self.head_dim} / {self.v_head_dim} do not fit the shared "
+                       f"memory of a CTA")
+        return out
+
+    def cache_need(self):
+        return PagedNeed(kv_heads=self.num_kv_heads, head_dim=self.k_row, window=self.window,
+                         v_head_dim=None if self.v_head_dim == self.k_row else self.v_head_dim)
+
+    def bind(self, params, rt) -> None:
+        import torch
+        super().bind(params, rt)
+        if not params:
+            return
+        if self.has_bias:
+            self.in_bias = torch.cat([self.q_bias, self.k_bias, self.v_bias]).contiguous()
+        if self.sink_kind == "zero":
+            self.sink = torch.zeros(self.num_heads, dtype=torch.float32, device=rt.device)
+
+    def core(self, proj, ctx, cache, out, out_scale: float = 1.0) -> None:
+        if out_scale != 1.0:
+            raise NotImplementedError("mixed-score attention takes no branch factor")
+        ops = self.rt.ops
+        gv = ctx.groups[cache.group]
+        if cache.write:
+            ops.paged_write_kv(proj[:, self.q_size:self.q_size + self.k_size], proj[:, self.q_size + self.k_size:],
+                               cache.k_pages, cache.v_pages, gv.slot_mapping)
+        ops.mixed_attention(proj[:, :self.q_size], cache.k_pages, cache.v_pages, gv.block_table, ctx, out, num_heads=self.num_heads,
+                            num_kv_heads=self.num_kv_heads, scale=self.scale, mix=self.talk, window=self.window, sink=self.sink)
+
+
+register_part("mixer", "mixed_score_attention", MixedScoreAttention)

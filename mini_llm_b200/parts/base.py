@@ -21,6 +21,8 @@ Interfaces (all tensors are CUDA tensors on the engine's stream):
                  (rotations), a no-op for absolute tables; ``max_positions``.
 * Embedding:     ``forward(ctx, positions_part) -> x_f32[T,D]``.
 * Head:          ``forward(y[R,D], ctx) -> logits_f32[R,V]``.
+* PassInput:     ``forward(x_f32[T,D], x0_f32[T,D], ctx, t) -> x``: makes the residual anew at the start of pass t of a
+                 looped stretch of layers, from what it was and the embedded rows x0.
 * Join:          ``forward(y_f32[T,D], x_f32[T,D], ctx)``: brings a branch's result y into the residual x
                  (a norm and a scale on y, say).  Mixers and feed-forwards with ``can_overwrite = True``
                  take ``accumulate=False`` and then write their result instead of adding it.
@@ -94,6 +96,13 @@ class Join(Part):
         raise NotImplementedError
 
 
+class PassInput(Part):
+    category = "pass_input"
+
+    def forward(self, x, x0, ctx, t):  # pragma: no cover
+        raise NotImplementedError
+
+
 class Positions(Part):
     category = "positions"
     max_positions: Optional[int] = None
@@ -122,7 +131,7 @@ class Head(Part):
 
 _REGISTRIES: Dict[str, Dict[str, Callable[..., Any]]] = {
     "norm": {}, "mixer": {}, "feed_forward": {}, "positions": {}, "embedding": {}, "head": {},
-    "arrangement": {}, "join": {},
+    "arrangement": {}, "join": {}, "pass_input": {},
 }
 
 

@@ -1,7 +1,8 @@
 """Joins: how a branch's result reaches the residual stream when that is more than a sum.
 
-``NormScaleJoin``: x += rms_norm(y, w) * s, the branch's result normed once more (plain weights, eps inside the
-root) and multiplied column by column by a learned scale before it is added; all 32-bit, one kernel.
+``NormScaleJoin``: x += rms_norm(y, w) * s * factor, the branch's result normed once more (plain weights, eps inside the
+root) and multiplied column by column by a learned scale (optional) and by a constant before it is added; all 32-bit, one
+kernel.
 
 ``PostNormJoin``: x <- rms_norm(alpha * x + y, w), the block that norms after the sum; the new x also comes back in the
 activation dtype for the branch that reads it next; all 32-bit, one kernel.
@@ -15,10 +16,11 @@ class NormScaleJoin(Join):
     norms_next = True       # forward(..., then_norm=) also norms the new x for the next branch
     takes_pairs = True      # forward(..., pairs=) takes the weighted sum over a routed feed-forward's choices itself
 
-    def __init__(self, hidden_size: int, eps: float, scaled: bool = True):
+    def __init__(self, hidden_size: int, eps: float, scaled: bool = True, factor: float = 1.0):
         self.hidden_size = int(hidden_size)
         self.eps = float(eps)
         self.scaled = bool(scaled)
+        self.factor = float(factor)
         self.scale = None
 
     def param_specs(self):
@@ -26,6 +28,11 @@ class NormScaleJoin(Join):
         if self.scaled:
             p["scale"] = ParamSpec((self.hidden_size,), "vector")
         return p
+
+    def bind(self, params, rt) -> None:
+        super().bind(params, rt)
+        if "weight" in params and self.factor != 1.0:       # the constant rides in the norm's weights
+            self.weight = (self.weight * self.factor).contiguous()
 
     def forward(self, y, x, ctx, pairs=None, then_norm=None):
         """x += n(y [+ the weighted pairs], w) * s.  ``pairs``: (results [T * top, D], weights [T, top], top) of a routed

@@ -47,21 +47,28 @@ GATE_ACTIVATIONS = ("relu", "silu", "gelu_tanh", "gelu_erf")
 
 
 class GatedMLP(FeedForward):
-    """x += W_down (act(W_gate h) * (W_up h)), no biases.  The gate and the up matrix are stacked into one
+    """x += W_down (act(W_gate h) * (W_up h)), with a bias on each of the three when ``bias``.  The gate and the up matrix are stacked into one
     [2F, D] matrix when the weights are bound, so both come from one product; a small kernel applies the
     activation and multiplies the halves; the down-projection adds into the residual in its epilogue."""
 
-    def __init__(self, hidden_size: int, inner_size: int, activation: str = "silu"):
+    def __init__(self, hidden_size: int, inner_size: int, activation: str = "silu", bias: bool = False):
         if activation not in GATE_ACTIVATIONS:
             raise ValueError(f"GatedMLP activation must be one of {GATE_ACTIVATIONS}, got {activation!r}")
         self.hidden_size = int(hidden_size)
         self.inner_size = int(inner_size)
         self.activation = activation
+        self.has_bias = bool(bias)
+        self.gate_up_bias = self.down_bias = None
 
     def param_specs(self):
-        return {"gate_weight": ParamSpec((self.inner_size, self.hidden_size), "matrix"),
-                "up_weight": ParamSpec((self.inner_size, self.hidden_size), "matrix"),
-                "down_weight": ParamSpec((self.hidden_size, self.inner_size), "matrix")}
+        p = {"gate_weight": ParamSpec((self.inner_size, self.hidden_size), "matrix"),
+             "up_weight": ParamSpec((self.inner_size, self.hidden_size), "matrix"),
+             "down_weight": ParamSpec((self.hidden_size, self.inner_size), "matrix")}
+        if self.has_bias:
+            p["gate_bias"] = ParamSpec((self.inner_size,), "vector")
+            p["up_bias"] = ParamSpec((self.inner_size,), "vector")
+            p["down_bias"] = ParamSpec((self.hidden_size,), "vector")
+        return p
 
     def bind(self, params, rt) -> None:
         import torch
@@ -70,6 +77,8 @@ class GatedMLP(FeedForward):
             self.gate_up_weight = torch.cat([self.gate_weight, self.up_weight], 0).contiguous()
             self.gate_weight = self.gate_up_weight[:self.inner_size]
             self.up_weight = self.gate_up_weight[self.inner_size:]
+        if "gate_bias" in params:
+            self.gate_up_bias = torch.cat([self.gate_bias, self.up_bias]).contiguous()
 
     accepts_lazy_norm = True
     can_overwrite = True                # forward(..., accumulate=False) writes the result instead of adding it
@@ -78,14 +87,14 @@ class GatedMLP(FeedForward):
         """The first half: gate | up of h (a tensor or a norm not yet evaluated).  It only reads; an arrangement whose
         branches all read the same x calls it before any branch adds to x."""
         gu = ctx.ws.buf("ff_gate_up", h.shape[0], 2 * self.inner_size, self.rt.act_dtype)
-        self.rt.ops.linear(h, self.gate_up_weight, None, out=gu)
+        self.rt.ops.linear(h, self.gate_up_weight, self.gate_up_bias, out=gu)
         return gu
 
     def finish(self, gu, ctx, out_accum, accumulate: bool = True):
         ops = self.rt.ops
         mid = ctx.ws.buf("ff_mid", gu.shape[0], self.inner_size, self.rt.act_dtype)
         ops.gated_act(gu, mid, self.activation)
-        ops.linear(mid, self.down_weight, None, out=out_accum, accumulate=accumulate)
+        ops.linear(mid, self.down_weight, self.down_bias, out=out_accum, accumulate=accumulate)
 
     def forward(self, h, ctx, out_accum, accumulate: bool = True):
         self.finish(self.project(h, ctx), ctx, out_accum, accumulate)

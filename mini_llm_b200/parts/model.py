@@ -50,6 +50,7 @@ class Model:
         self.spec = spec
         self.embedding = build_part("embedding", spec.embedding)
         self.positions = build_part("positions", spec.positions)
+        self.pass_input = build_part("pass_input", spec.pass_input) if spec.pass_input is not None else None
         self.layers: List[Layer] = [Layer(ls, spec.hidden_size) for ls in spec.layers]
         self.final_norm = build_part("norm", spec.final_norm)
         self.head = build_part("head", spec.head)
@@ -112,6 +113,8 @@ class Model:
         or None when no logits are wanted."""
         x = self.embedding.forward(ctx, self.positions)
         for entry, cache in zip(self.spec.schedule, self._caches):
+            if entry.enters_pass is not None:
+                x = self.pass_input.forward(x, self.embedding.kept(ctx), ctx, entry.enters_pass)
             layer = self.layers[entry.layer]
             x = layer.arrangement(layer, x, ctx, cache)
         if ctx.R == 0:

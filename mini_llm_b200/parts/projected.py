@@ -29,6 +29,8 @@ class ProjectedMixer(Mixer):
     in_names: Sequence[str] = ()        # parameters stacked (by rows) into the input projection, in this order
     out_name: str = "out_weight"        # the output projection [hidden, core_width]
     in_bias = None                      # a bias on the input projection (float32 [in_width]), set at bind by a mixer that has one
+    out_bias = None                     # a bias on the output projection (float32 [hidden]); a mixer that has one runs alone, not as a branch
+    proj_f32 = False                    # the projected columns are handed to the core in 32-bit whatever the engine's dtype
 
     @property
     def in_width(self) -> int:
@@ -52,11 +54,12 @@ class ProjectedMixer(Mixer):
         ops = self.rt.ops
         T = h.shape[0]
         n_in = self.in_weight.shape[0]
-        proj = ctx.ws.buf("mix_proj", T, -(-n_in // 8) * 8, self.rt.act_dtype)[:, :n_in]    # rows stay 16-byte aligned
+        proj = ctx.ws.buf("mix_proj", T, -(-n_in // 8) * 8,
+                          torch.float32 if self.proj_f32 else self.rt.act_dtype)[:, :n_in]  # rows stay 16-byte aligned
         ops.linear(h, self.in_weight, self.in_bias, out=proj)
         mid = ctx.ws.buf("mix_core", T, self.core_width, self.rt.act_dtype)
         self.core(proj, ctx, cache, mid)
-        ops.linear(mid, getattr(self, self.out_name), None, out=out_accum, accumulate=accumulate)
+        ops.linear(mid, getattr(self, self.out_name), self.out_bias, out=out_accum, accumulate=accumulate)
 
 
 class ParallelMixer(Mixer):

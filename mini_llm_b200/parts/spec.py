@@ -72,13 +72,15 @@ class ScheduleEntry:
     and writes nothing to it.  ``private_cache``: the run has a cache and a state
     of its own (of the kind its layer's mixer needs) that no other run touches:
     a layer that runs several times with the same weights, each run with its own
-    history.  ``cache_unit`` (set by ModelSpec) is the id under which the cache
+    history.  ``enters_pass`` t: before this run the model's ``pass_input`` part makes the residual anew for pass t of a
+    looped stretch.  ``cache_unit`` (set by ModelSpec) is the id under which the cache
     manager keeps the run's cache: the layer's index, or a number beyond the
     layers for a private one."""
 
     layer: int
     cache_of: Optional[int] = None
     private_cache: bool = False
+    enters_pass: Optional[int] = None
     cache_unit: Optional[int] = None
 
     def __post_init__(self):
@@ -98,6 +100,7 @@ class ModelSpec:
     final_norm: PartSpec
     head: PartSpec
     schedule: Optional[List[ScheduleEntry]] = None
+    pass_input: Optional[PartSpec] = None    # category "pass_input": runs before every entry that enters a pass
     max_positions: Optional[int] = None      # None: the position encoding sets no limit
     eos_token_id: Optional[int] = None
     ignored_tensors: List[str] = field(default_factory=list)   # regexes of checkpoint tensors to skip
@@ -106,6 +109,8 @@ class ModelSpec:
         if self.schedule is None:
             self.schedule = [ScheduleEntry(i) for i in range(len(self.layers))]
         n = len(self.layers)
+        if self.pass_input is None and any(e.enters_pass is not None for e in self.schedule):
+            raise ValueError("the schedule enters a pass but the model names no pass_input part")
         private = 0
         for e in self.schedule:
             if not (0 <= e.layer < n) or not (0 <= e.cache_of < n):
@@ -120,6 +125,8 @@ class ModelSpec:
         """(label, PartSpec) of every part, in a fixed order."""
         yield "embedding", self.embedding
         yield "positions", self.positions
+        if self.pass_input is not None:
+            yield "pass_input", self.pass_input
         for i, l in enumerate(self.layers):
             if l.mixer_norm is not None:
                 yield f"layers.{i}.mixer_norm", l.mixer_norm
