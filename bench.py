@@ -40,8 +40,8 @@ with "impl": "reference" and "dtype": "fp32".  The reference holds at most 16 re
 (more are cut) and there is no batch-64 point.  Where it cannot be built or run the line is
 {"impl": "reference", "unavailable": "<why>"}.
 
-``--compare-designs [small,medium,large]`` measures the engine's other designs, Finuvik, Falisun, Mumopel and Kusirax, beside
-GPT-2 at equal width, depth and head count (bfloat16 unless --dtype is given; ``--designs gpt2,falisun`` picks some).
+``--compare-designs [small,medium,large]`` measures the engine's other designs, Finuvik, Falisun, Mumopel, Kusirax and Zadenex,
+beside GPT-2 at equal width, depth and head count (bfloat16 unless --dtype is given; ``--designs gpt2,falisun`` picks some).
 
 ``--profile-step prefill|decode [--kernel-times]`` runs one small eager step (for a profiler, or to
 print each kernel's share of the step from CUDA events); ``--workload medium|xl`` runs the
@@ -316,9 +316,11 @@ def profile_step(kind: str, dtype: str, layers: int, batch: int, kernel_times: b
     from mini_llm_b200.engine.runner import ModelRunner, StepEntry
 
     cfg = dict(SMALL, n_layer=layers)
-    if design in ("finuvik", "falisun", "mumopel", "kusirax"):  # the same step of the other designs at the "small" comparison size
+    if design in ("finuvik", "falisun", "mumopel", "kusirax", "zadenex"):  # the same step of the other designs at the "small" comparison size
         cfg = design_configs("small")[design]
         cfg["layers"] = cfg["layers"][:layers]
+        if cfg.get("loop") and cfg["loop"]["stop"] > layers:
+            cfg["loop"] = None
         cfg["n_positions"], cfg["vocab_size"] = DESIGN_POSITIONS, cfg["vocab"]      # the names used below
     times = None
     with tempfile.TemporaryDirectory(prefix="mini_llm_prof_") as d:
@@ -502,7 +504,25 @@ def design_configs(size: str):
             dict(kind="moe", router=dict(experts=8, top=2, scale=2.0, groups=dict(count=4, keep=2)), expert=dict(ff=3 * F // 8 // 8 * 8))
         kl.append(dict(type=kind, mixer=mixer, mlp=mlp))
     kusirax = dict(architecture="Kusirax", width=D, vocab=DESIGN_VOCAB, norm=dict(eps=1e-5), postln_alpha=2.0, layers=kl)
-    return {"gpt2": gpt2, "finuvik": finuvik, "falisun": falisun, "mumopel": mumopel, "kusirax": kusirax}
+    # Zadenex at the same width, heads and key/value heads: latent attention (Falisun's sizes, queries through a latent of half
+    # the width), a matrix memory (heads of 64 x 64 over the whole width, as Kusirax's recurrence), attention with mixed scores
+    # over the last 768 tokens, a matrix memory again (large: latent attention, matrix memory); dense feed-forwards of Finuvik's
+    # inner size; the second layer is a looped stretch of one pass, so that a pass's input product is part of the step
+    kinds = ["latent_attention", "mlstm", "attention", "mlstm"]
+    zl = []
+    for i in range(L):
+        kind = kinds[i % len(kinds)]
+        if kind == "mlstm":
+            mixer = dict(heads=D // 64, dim=64, vdim=64, gate_cap=15.0)
+        elif kind == "attention":
+            mixer = dict(heads=H, kv_heads=z["kv_heads"], dim=dh, vdim=dh, scale=dh ** -0.5, mask=dict(size=768))
+        else:
+            mixer = dict(heads=H, dim=dh, rot_dim=dh // 2, vdim=dh, kv_rank=rank, q_rank=D // 2, scale=(dh + dh // 2) ** -0.5,
+                         rot=dict(base=10000.0, dims=dh // 2))
+        zl.append(dict(type=kind, mixer=mixer, mlp=dict(kind="dense", ff=F)))
+    zadenex = dict(architecture="Zadenex", width=D, vocab=DESIGN_VOCAB, norm=dict(eps=1e-5), embedding=dict(scale=4.0),
+                   residual_mult=0.5, loop=dict(start=1, stop=2, times=1), layers=zl)
+    return {"gpt2": gpt2, "finuvik": finuvik, "falisun": falisun, "mumopel": mumopel, "kusirax": kusirax, "zadenex": zadenex}
 
 
 def _design_model(model_dir, dtype, batch, tokens):
@@ -607,7 +627,7 @@ def design_decode(model_dir, dtype, batch, steps):
 
 
 def run_compare_designs(sizes, dtype: str, batch: int, steps: int, designs=None) -> int:
-    """Prefill and decode throughput of Finuvik, Falisun and Mumopel beside GPT-2 at equal width, depth and head count, random
+    """Prefill and decode throughput of the other designs beside GPT-2 at equal width, depth and head count, random
     weights; one JSON line per size.  Per kernel entry point the line carries the
     microseconds of one eager step, from which the rooflines of the like kernels are compared."""
     import torch
@@ -765,7 +785,7 @@ def main() -> int:
     ap.add_argument("--no-points", action="store_true", help="skip the batch 1 / 64, prefill and other-precision measurements")
     ap.add_argument("--profile-step", choices=["prefill", "decode"],
                     help="run one small eager step for a profiler instead of the benchmark")
-    ap.add_argument("--design", choices=["gpt2", "finuvik", "falisun", "mumopel", "kusirax"], default="gpt2",
+    ap.add_argument("--design", choices=["gpt2", "finuvik", "falisun", "mumopel", "kusirax", "zadenex"], default="gpt2",
                     help="with --profile-step: the model whose step is run (the other designs: the 'small' size of --compare-designs)")
     ap.add_argument("--kernel-times", action="store_true",
                     help="with --profile-step: time every launch of one eager step with CUDA events and print the shares")
@@ -776,7 +796,7 @@ def main() -> int:
     ap.add_argument("--compare-designs", nargs="?", const="small,medium,large", metavar="SIZES",
                     help="measure Finuvik, Falisun and Mumopel beside GPT-2 at equal sizes (a comma list of small, medium, large) "
                          "instead of the benchmark: prefill of 2 x 1024 tokens and decode at --batch, one JSON line per size")
-    ap.add_argument("--designs", default="", help="with --compare-designs: a comma list of gpt2, finuvik, falisun, mumopel, kusirax (default: all)")
+    ap.add_argument("--designs", default="", help="with --compare-designs: a comma list of gpt2, finuvik, falisun, mumopel, kusirax, zadenex (default: all)")
     args = ap.parse_args()
     if args.compare_designs:
         sizes = [z for z in args.compare_designs.split(",") if z]

@@ -10,9 +10,9 @@
 //
 // Three kernels.  `step`: steps of single tokens in one launch, one CTA per (request, head).  `scan` and `finish`: steps that
 // carry prompt portions.  `scan`: a CTA takes COLS columns of one (request, head)'s S; thread (column, row group) keeps WR
-// rows in registers for the whole walk; tokens come 16 at a time (q, k, v by cp.async, two buffers); one more warp makes the
-// gates a chunk ahead (a lane per token; only m runs token by token) and, in the first column block, walks n and takes
-// n . q; the row groups' partial outputs meet in group order.  Every element of S and n is a recurrence of its own and m runs
+// rows in registers for the whole walk; tokens come 16 at a time (q, k, v by cp.async, two buffers); a warp of its own makes
+// the gates a chunk ahead (a lane per token; only m runs token by token), and in the first column block further warps walk n
+// and take n . q; the row groups' partial outputs meet in group order.  Every element of S and n is a recurrence of its own and m runs
 // token by token, so the state after some tokens is the same bits however they were cut into steps.  `finish`: a warp per
 // (token, head): the denominator, the unit norm, the weight and the gate.
 #include "common.cuh"
@@ -48,18 +48,20 @@ __device__ __forceinline__ void cp16(float* dst, const float* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(d), "l"(src) : "memory");
 }
 
-// grid (requests, heads, column blocks), block COLS * G threads rounded up to whole warps + 32, G = ceil(dk / WR) row groups;
-// the last warp is the gates' and n's.  raw [T][H * dv]: S^T q (q not yet scaled); aux [T][H][2]: n . q and m.  vec: rows can be copied 16 bytes at
-// a time.
+// grid (requests, heads, column blocks).  Block: COLS * G threads (G = ceil(dk / WR) row groups) rounded up to whole warps,
+// the gates' warp, then NW = ceil(dk / 32) warps that walk n (a lane per row; the first column block only).
+// raw [T][H * dv]: S^T q (q not yet scaled); aux [T][H][2]: n . q and m.  vec: rows can be copied 16 bytes at a time.
 template <int WR, int COLS>
-__global__ void __launch_bounds__(COLS * 16 + 32)
+__global__ void __launch_bounds__(COLS * 16 + 32 + WR * 16)
 mlstm_scan_kernel(float* __restrict__ raw, float* __restrict__ aux, int vec, MlstmArgs a) {
     extern __shared__ __align__(16) float sm[];
     const int dk = a.dk, dv = a.dv, H = a.H;
-    const int G = (dk + WR - 1) / WR, np = G * WR, nmain = G * COLS;       // rows beyond dk are zeros
+    const int G = (dk + WR - 1) / WR, NW = (dk + 31) / 32, nmain = G * COLS;
+    const int np = max(G * WR, NW * 32);        // rows beyond dk are zeros
     const int buf_floats = CH * (2 * np + COLS);
     float* os = sm + 2 * buf_floats;            // [G][CH][COLS]
-    float* gs = os + G * CH * COLS;             // [2][2][CH]: a and b of two chunks
+    float2* gs = reinterpret_cast<float2*>(os + G * CH * COLS);      // [2][CH]: (a, b) of two chunks
+    float* ns = reinterpret_cast<float*>(gs + 2 * CH);               // [NW][CH]: n . q of the chunk, per warp of rows
     pdl_wait();
     pdl_launch();
     const int seq = blockIdx.x, h = blockIdx.y, j0 = blockIdx.z * COLS;
@@ -70,11 +72,12 @@ mlstm_scan_kernel(float* __restrict__ raw, float* __restrict__ aux, int vec, Mls
     float* Sg = st + (size_t)h * dk * dv;
     float* ng = st + (size_t)H * dk * dv + (size_t)h * dk;
     float* mg = st + (size_t)H * dk * (dv + 1) + h;
-    const bool gate_warp = tid >= nthreads - 32, main_thread = tid < nmain;
-    const int lane = tid & 31;
+    const int gate0 = (nmain + 31) / 32 * 32, lane = tid & 31, aw = (tid - gate0) >> 5;      // aw: 0 the gates' warp, 1 .. NW those of n
+    const bool main_thread = tid < nmain, gate_warp = tid >= gate0 && aw == 0, keeps_n = blockIdx.z == 0;
+    const bool n_warp = tid >= gate0 && aw > 0 && keeps_n;
+    const int nrow = (aw - 1) * 32 + lane;      // an n warp's row
     const int col = tid % COLS, g = tid / COLS, j = j0 + col;
     const bool live = main_thread && j < dv;
-    const bool keeps_n = blockIdx.z == 0;
     // padded rows of q and k in both buffers are zero and stay zero
     for (int i = tid; i < 2 * CH * (np - dk); i += nthreads) {
         const int r = i % (np - dk), c = (i / (np - dk)) % CH, b = i / ((np - dk) * CH);
@@ -114,7 +117,7 @@ mlstm_scan_kernel(float* __restrict__ raw, float* __restrict__ aux, int vec, Mls
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    float m = 0.f;                              // the gate warp's running maximum
+    float m = 0.f;                              // the gates' warp: the running maximum
     float zi = 0.f, zf = 0.f;                   // its next chunk's gate projections, a lane per token
     auto fetch_gates = [&](int c0) {
         if (lane < min(CH, n - c0)) {
@@ -137,30 +140,25 @@ mlstm_scan_kernel(float* __restrict__ raw, float* __restrict__ aux, int vec, Mls
             }
         }
         if (lane < nc) {
-            gs[buf * 2 * CH + lane] = expf(before - after);
-            gs[buf * 2 * CH + CH + lane] = expf(li - after);
+            gs[buf * CH + lane] = make_float2(expf(before - after), expf(li - after));
             if (keeps_n) aux[((size_t)(t0 + c0 + lane) * H + h) * 2 + 1] = after;
         }
     };
     stage(0, 0);
-    float s[WR], nr[MAX_D / 32];
+    float s[WR];                                // a main thread's rows of its column; an n warp's row in s[0]
+#pragma unroll
+    for (int i = 0; i < WR; ++i) s[i] = 0.f;
     if (gate_warp) {
         m = *mg;
         fetch_gates(0);
         make_gates(0, 0);
         if (CH < n) fetch_gates(CH);
+    } else if (n_warp) {
+        if (nrow < dk) s[0] = ng[nrow];
+    } else if (live) {
 #pragma unroll
-        for (int i = 0; i < MAX_D / 32; ++i) {
-            const int r = lane + 32 * i;
-            nr[i] = (keeps_n && r < dk) ? ng[r] : 0.f;
-        }
-    }
-    if (main_thread) {
-#pragma unroll
-        for (int i = 0; i < WR; ++i) {
-            const int r = g * WR + i;
-            s[i] = (live && r < dk) ? Sg[(size_t)r * dv + j] : 0.f;
-        }
+        for (int i = 0; i < WR; ++i)
+            if (g * WR + i < dk) s[i] = Sg[(size_t)(g * WR + i) * dv + j];
     }
     for (int c0 = 0, buf = 0; c0 < n; c0 += CH, buf ^= 1) {
         const int nc = min(CH, n - c0);
@@ -171,10 +169,11 @@ mlstm_scan_kernel(float* __restrict__ raw, float* __restrict__ aux, int vec, Mls
         const float* qd = sm + buf * buf_floats;
         const float* kd = qd + CH * np;
         const float* vd = kd + CH * np;
-        const float* ga = gs + buf * 2 * CH;
+        const float2* ga = gs + buf * CH;
         if (main_thread) {
-            for (int c = 0; c < nc; ++c) {
-                const float at = ga[c], bv = ga[CH + c] * vd[c * COLS + col];
+            auto walk = [&](int c) {
+                const float2 ab = ga[c];
+                const float at = ab.x, bv = ab.y * vd[c * COLS + col];
                 const float4* q4 = reinterpret_cast<const float4*>(qd + c * np + g * WR);
                 const float4* k4 = reinterpret_cast<const float4*>(kd + c * np + g * WR);
                 float acc0 = 0.f, acc1 = 0.f;
@@ -191,35 +190,41 @@ mlstm_scan_kernel(float* __restrict__ raw, float* __restrict__ aux, int vec, Mls
                     acc1 = fmaf(s[4 * i + 3], q.w, acc1);
                 }
                 os[(g * CH + c) * COLS + col] = acc0 + acc1;
+            };
+            if (nc == CH) {
+#pragma unroll 4
+                for (int c = 0; c < CH; ++c) walk(c);
+            } else {
+                for (int c = 0; c < nc; ++c) walk(c);
             }
         } else if (gate_warp) {
-            if (keeps_n) {
-                float part[CH];
-#pragma unroll
-                for (int c = 0; c < CH; ++c) {
-                    part[c] = 0.f;
-                    if (c < nc) {
-                        const float at = ga[c], bt = ga[CH + c];
-#pragma unroll
-                        for (int i = 0; i < MAX_D / 32; ++i) {
-                            const int r = lane + 32 * i;
-                            if (r < dk) {
-                                nr[i] = fmaf(at, nr[i], bt * kd[c * np + r]);
-                                part[c] = fmaf(nr[i], qd[c * np + r], part[c]);
-                            }
-                        }
-                    }
-                }
-#pragma unroll
-                for (int c = 0; c < CH; ++c) {
-                    const float nq = warp_sum(part[c]);
-                    if (lane == c && c < nc) aux[((size_t)(t0 + c0 + c) * H + h) * 2] = nq;
-                }
-            }
             if (more) {
                 make_gates(c0 + CH, buf ^ 1);
                 if (c0 + 2 * CH < n) fetch_gates(c0 + 2 * CH);
             }
+        } else if (n_warp) {
+            float part[CH];
+#pragma unroll
+            for (int c = 0; c < CH; ++c) {
+                part[c] = 0.f;
+                if (c < nc) {
+                    const float2 ab = ga[c];
+                    s[0] = fmaf(ab.x, s[0], ab.y * kd[c * np + nrow]);
+                    part[c] = s[0] * qd[c * np + nrow];
+                }
+            }
+            // sums of 16 tokens over 32 lanes: at every step a lane keeps half of its tokens and hands the other half over
+#pragma unroll
+            for (int w = CH / 2; w >= 1; w /= 2) {
+                const bool up = lane & w;
+#pragma unroll
+                for (int i = 0; i < w; ++i) {
+                    const float keep = up ? part[i + w] : part[i], give = up ? part[i] : part[i + w];
+                    part[i] = keep + __shfl_xor_sync(0xffffffffu, give, w);
+                }
+            }
+            part[0] += __shfl_xor_sync(0xffffffffu, part[0], 16);
+            if (lane < CH) ns[(aw - 1) * CH + lane] = part[0];       // lane l < 16 ends with token l
         }
         __syncthreads();
         for (int i = tid; i < nc * COLS; i += nthreads) {       // the row groups meet in group order
@@ -229,22 +234,19 @@ mlstm_scan_kernel(float* __restrict__ raw, float* __restrict__ aux, int vec, Mls
             for (int gg = 1; gg < G; ++gg) acc += os[(gg * CH + c) * COLS + d];
             raw[(size_t)(t0 + c0 + c) * ((size_t)H * dv) + (size_t)h * dv + j0 + d] = acc;
         }
+        if (n_warp && aw == 1 && lane < nc) {
+            float nq = ns[lane];
+            for (int w = 1; w < NW; ++w) nq += ns[w * CH + lane];
+            aux[((size_t)(t0 + c0 + lane) * H + h) * 2] = nq;
+        }
     }
     if (!a.write_state) return;
     if (live) {
 #pragma unroll
-        for (int i = 0; i < WR; ++i) {
-            const int r = g * WR + i;
-            if (r < dk) Sg[(size_t)r * dv + j] = s[i];
-        }
+        for (int i = 0; i < WR; ++i)
+            if (g * WR + i < dk) Sg[(size_t)(g * WR + i) * dv + j] = s[i];
     }
-    if (gate_warp && keeps_n) {
-#pragma unroll
-        for (int i = 0; i < MAX_D / 32; ++i) {
-            const int r = lane + 32 * i;
-            if (r < dk) ng[r] = nr[i];
-        }
-    }
+    if (n_warp && nrow < dk) ng[nrow] = s[0];
     // m is written by mlstm_finish_kernel: every column block of this launch reads it
 }
 
@@ -410,10 +412,10 @@ MLLM_EXPORT int mllm_mlstm_scan(const float* proj, long long ld, int q_off, int 
     // every CTA is one chain of dependent token steps: narrower CTAs shorten it as long as they all run at once
     const int cols = want_cols ? want_cols : ((dv > 16 && (long long)S * H * ((dv + 15) / 16) <= sms) ? 16 : 32);
     const int WR = dk <= 64 ? 4 : (dk <= 128 ? 8 : 16);
-    const int G = (dk + WR - 1) / WR, np = G * WR;
-    const size_t smem = sizeof(float) * (2 * (size_t)CH * (2 * np + cols) + (size_t)G * CH * cols + 4 * CH);
+    const int G = (dk + WR - 1) / WR, NW = (dk + 31) / 32, np = G * WR > NW * 32 ? G * WR : NW * 32;
+    const size_t smem = sizeof(float) * (2 * (size_t)CH * (2 * np + cols) + (size_t)G * CH * cols + 4 * CH + (size_t)NW * CH);
     const int vec = dk % 4 == 0 && dv % 4 == 0 && ld % 4 == 0 && q_off % 4 == 0 && k_off % 4 == 0 && v_off % 4 == 0 && (uintptr_t)proj % 16 == 0;
-    const dim3 grid(S, H, (dv + cols - 1) / cols), block((cols * G + 31) / 32 * 32 + 32);
+    const dim3 grid(S, H, (dv + cols - 1) / cols), block((cols * G + 31) / 32 * 32 + 32 + 32 * NW);
 #define MLLM_SCAN(WRR, CC)                                                                                               \
     do {                                                                                                                 \
         if (smem > 48 * 1024)                                                                                            \
