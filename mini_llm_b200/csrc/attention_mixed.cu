@@ -404,16 +404,31 @@ attention_mixed_mma_kernel(const __nv_bfloat16* q, const __nv_bfloat16* k_pages,
     const int* bt = a.bt + (size_t)seq * a.bt_stride;
     const int first_key = first_visible(a.window, pos0);
     const int kp8 = dk / 8, vp8 = dv / 8;
+    // A key's row of one key/value head (its kp8 + vp8 pieces of 16 bytes) is copied by `1 << lsh` lanes, so a thread's key,
+    // head and pieces follow from shifts; lane l of a warp has looked up the page row of key l of the tile.
+    const int per = kp8 + vp8, lsh = per <= 4 ? 2 : (per <= 8 ? 3 : (per <= 16 ? 4 : 5));
+    const int ps_shift = (a.ps & (a.ps - 1)) == 0 ? __ffs(a.ps) - 1 : -1;       // pages of a power of two: shifts
     auto stage = [&](int j, int buf) {                           // key tile j into buffer buf
         bf* kd = Ks + (size_t)buf * G * MK * qrow;
         bf* vd = Vs + (size_t)buf * G * MK * vrow;
-        const int per = kp8 + vp8;
-        for (int i = tid; i < MK * G * per; i += NT) {
-            const int piece = i % per, gk = i / per, g = gk % G, key = gk / G, kp = j * MK + key;
-            const bool ok = kp <= pos_max && kp >= first_key;
-            const size_t rn = ok ? ((size_t)bt[kp / a.ps] * G + g) * a.ps + kp % a.ps : 0;
-            if (piece < kp8) cp_async16(kd + ((size_t)g * MK + key) * qrow + piece * 8, k_pages + rn * dk + piece * 8, ok);
-            else cp_async16(vd + ((size_t)g * MK + key) * vrow + (piece - kp8) * 8, v_pages + rn * dv + (piece - kp8) * 8, ok);
+        int mine = -1;
+        {
+            const int kp = j * MK + lane;
+            if (kp <= pos_max && kp >= first_key) {
+                const int pg = ps_shift >= 0 ? kp >> ps_shift : kp / a.ps;
+                const int off = ps_shift >= 0 ? kp & (a.ps - 1) : kp % a.ps;
+                mine = bt[pg] * G * a.ps + off;
+            }
+        }
+        for (int r = tid >> lsh; r < MK * G; r += NT >> lsh) {   // row r: key r & 31 of head r >> 5 (the same trips for a whole warp)
+            const int key = r & (MK - 1), g = r >> 5;
+            const int row0 = __shfl_sync(0xffffffffu, mine, key);
+            const bool ok = row0 >= 0;
+            const size_t rn = ok ? (size_t)row0 + (size_t)g * a.ps : 0;
+            for (int piece = lane & ((1 << lsh) - 1); piece < per; piece += 1 << lsh) {
+                if (piece < kp8) cp_async16(kd + (size_t)r * qrow + piece * 8, k_pages + rn * dk + piece * 8, ok);
+                else cp_async16(vd + (size_t)r * vrow + (piece - kp8) * 8, v_pages + rn * dv + (piece - kp8) * 8, ok);
+            }
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };

@@ -331,7 +331,9 @@ class MixedScoreAttention(ProjectedMixer):
     three input projections have biases; ``out_bias``: so has the output projection.  ``sink``: "zero" (one is added to the
     softmax's denominator: a sink whose score is 0), "learned" (exp of a trained scalar per head is) or None.
 
-    Every head needs the raw scores of all the others, so a CTA of the kernels takes all heads of its queries."""
+    Every head needs the raw scores of all the others, so a CTA of the kernels takes all heads of its queries.  Where keys and
+    values have one size (a multiple of 8, so key rows have no padding) the input product writes them to their page slots from
+    its epilogue, as ``Attention`` does."""
 
     in_names = ("q_weight", "k_weight", "v_weight")
     out_name = "out_weight"
@@ -403,13 +405,27 @@ class MixedScoreAttention(ProjectedMixer):
     def core(self, proj, ctx, cache, out, out_scale: float = 1.0) -> None:
         if out_scale != 1.0:
             raise NotImplementedError("mixed-score attention takes no branch factor")
-        ops = self.rt.ops
-        gv = ctx.groups[cache.group]
         if cache.write:
-            ops.paged_write_kv(proj[:, self.q_size:self.q_size + self.k_size], proj[:, self.q_size + self.k_size:],
-                               cache.k_pages, cache.v_pages, gv.slot_mapping)
-        ops.mixed_attention(proj[:, :self.q_size], cache.k_pages, cache.v_pages, gv.block_table, ctx, out, num_heads=self.num_heads,
-                            num_kv_heads=self.num_kv_heads, scale=self.scale, mix=self.talk, window=self.window, sink=self.sink)
+            self.rt.ops.paged_write_kv(proj[:, self.q_size:self.q_size + self.k_size], proj[:, self.q_size + self.k_size:],
+                                       cache.k_pages, cache.v_pages, ctx.groups[cache.group].slot_mapping)
+        self._attend(proj[:, :self.q_size], ctx, cache, out)
+
+    def _attend(self, q, ctx, cache, out) -> None:
+        self.rt.ops.mixed_attention(q, cache.k_pages, cache.v_pages, ctx.groups[cache.group].block_table, ctx, out,
+                                    num_heads=self.num_heads, num_kv_heads=self.num_kv_heads, scale=self.scale, mix=self.talk,
+                                    window=self.window, sink=self.sink)
+
+    def forward(self, h, ctx, cache, out_accum, accumulate: bool = True):
+        if not (cache.write and self.head_dim == self.v_head_dim == self.k_row):
+            super().forward(h, ctx, cache, out_accum, accumulate)
+            return
+        ops = self.rt.ops
+        T = h.shape[0]
+        q = ops.linear_qkv_cache(h, self.in_weight, self.in_bias, ctx.ws.buf("attn_q", T, self.q_size, self.rt.act_dtype),
+                                 cache.k_pages, cache.v_pages, ctx.groups[cache.group].slot_mapping, ctx.ws)
+        mid = ctx.ws.buf("mix_core", T, self.core_width, self.rt.act_dtype)
+        self._attend(q, ctx, cache, mid)
+        ops.linear(mid, self.out_weight, self.out_bias, out=out_accum, accumulate=accumulate)
 
 
 register_part("mixer", "mixed_score_attention", MixedScoreAttention)
