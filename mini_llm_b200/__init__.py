@@ -1,5 +1,5 @@
-"""mini_llm_b200: a small, whole inference engine for one B200 (sm_100a): GPT-2, Finuvik, Falisun, Mumopel, Kusirax
-and Zadenex.
+"""mini_llm_b200: a small, whole inference engine for one B200 (sm_100a): GPT-2, Finuvik, Falisun, Mumopel, Kusirax,
+Zadenex and Zanelorn.
 
 Configuration and registry (``config``), safetensors weights (``weights``), model
 parts and their assembly (``parts``, ``models``), paged cache manager (``cache``),
@@ -9,9 +9,9 @@ hand-written CUDA kernels (``csrc``, reached through ``ops``).
 from .config.base import (ConfigError, EngineConfig, config_from_dict, load_config, register_architecture,
                           registered_architectures)
 from .parts import (attention, block, embedding, head, hyper, join, latent, mlp, mlstm, moe, norm, passes,  # noqa: F401
-                    positions, projected, recurrent, ssm, wkv)                                                     # (register the parts)
+                    positions, projected, recurrent, retention, side, ssm, wkv)                                    # (register the parts)
 from .parts.base import register_part
-from .models import falisun, finuvik, gpt2, kusirax, mumopel, zadenex  # noqa: F401  (register GPT2LMHeadModel, Finuvik, Falisun, Mumopel, Kusirax, Zadenex)
+from .models import falisun, finuvik, gpt2, kusirax, mumopel, zadenex, zanelorn  # noqa: F401  (register GPT2LMHeadModel, Finuvik, Falisun, Mumopel, Kusirax, Zadenex, Zanelorn)
 from .weights.random_init import write_random_model
 from .sampling.params import SamplingParams
 from .engine.request import Request, RequestState, Response

@@ -33,6 +33,7 @@ class PagedNeed:
     v_head_dim: Optional[int] = None  # size of a value row when it differs from a key row's (None: head_dim)
     values_in_keys: bool = False      # a token's value is a part of its key row (a cache of latents): no value pool
     chunk: Optional[int] = None       # a query sees only keys of its own block of ``chunk`` positions (counted from 0)
+    keep_first: int = 0               # with a window or a chunk: the first tokens that stay visible all the same
 
     @property
     def value_dim(self) -> int:
@@ -226,7 +227,8 @@ class CacheManager:
             first_needed = first_key // self.page_size
             tab = g.tables[req]
             gone = []
-            for p in range(lv.first_kept[g.index], min(first_needed, len(tab))):
+            kept = self.pages_for(g.need.keep_first)        # pages with tokens that every later query sees
+            for p in range(max(lv.first_kept[g.index], kept), min(first_needed, len(tab))):
                 if tab[p] != RELEASED:
                     gone.append(tab[p])
                     tab[p] = RELEASED

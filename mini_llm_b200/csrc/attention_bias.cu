@@ -13,7 +13,10 @@
 // (`softcap` c > 0), and a linear distance penalty slope_h * (i - j) taken off the score (`slopes`, a number per head;
 // the product of the slope and the distance is taken in 32-bit in the kernel, so it needs no table and no bound on the
 // context).
-// Either table, the slopes, the cap, the window, the chunk and the sink may be absent.
+// `keep_first` f: the first f positions of the request stay visible beyond the window or the chunk (key tiles that lie
+// wholly between them and the window are not visited).  `gate`: the output is multiplied, entry by entry, with
+// sigmoid(gate[t][h * dv + d]) before it is rounded.
+// Either table, the slopes, the cap, the window, the chunk, the sink, the kept keys and the gate may be absent.
 // Scores, biases, softmax and the weighted sum are 32-bit (expf, not the fast intrinsic) for both cache dtypes.
 //
 // Four kernels (the fourth, `mma`, is described where it stands).  `simt`: one warp per (token, head), 32 keys at a time: any step, and the plain twin of the
@@ -54,6 +57,9 @@ struct BiasArgs {
     const float* sink;          // [H] or null: exp(sink[h]) joins the softmax denominator
     float softcap;              // > 0: the scaled product s becomes softcap * tanh(s / softcap) before the biases
     const float* slopes;        // [H] or null: slopes[h] * (i - j) is taken off the score
+    int keep;                   // the first `keep` positions stay visible
+    const void* gate;           // [T][gate_stride] in the dtype of q, or null
+    long long gate_stride;
 };
 
 // the cap on a scaled product (before any bias)
@@ -65,6 +71,19 @@ __device__ __forceinline__ int first_visible(const BiasArgs& a, int p) {
     if (a.window > 0 && p - a.window + 1 > 0) first = p - a.window + 1;
     if (a.chunk > 0) first = max(first, (p / a.chunk) * a.chunk);
     return first;
+}
+
+// whether the query at p sees the key at kp, given kp <= p and first = first_visible(p)
+__device__ __forceinline__ bool sees(const BiasArgs& a, int kp, int first) { return kp >= first || kp < a.keep; }
+
+// whether no query from the one with first_visible = first on sees a key of [k_lo, k_hi]
+__device__ __forceinline__ bool in_gap(const BiasArgs& a, int k_lo, int k_hi, int first) { return k_lo >= a.keep && k_hi < first; }
+
+template <typename T>
+__device__ __forceinline__ float gate_of(const BiasArgs& a, int t, int col) {
+    if (!a.gate) return 1.0f;
+    const float g = to_f32(reinterpret_cast<const T*>(a.gate)[(size_t)t * a.gate_stride + col]);
+    return 1.0f / (1.0f + expf(-g));
 }
 
 // One warp walks the keys [k_lo, k_hi] (inclusive, absolute positions) of one (token, head) in chunks of 32 that
@@ -145,13 +164,15 @@ attention_bias_simt_kernel(const T* q, long long q_stride, const T* k_pages, con
     for (int i = 0; i < NACC; ++i) acc[i] = 0.f;
     float m = -INFINITY, l = 0.f;
     if (a.sink) { m = a.sink[h]; l = 1.f; }
+    if (a.keep > 0 && first > 0)                             // the kept keys before the window
+        warp_walk<T>(qs[warp], k_pages, v_pages, bt, p, h, hk, Hkv, dk, dv, page_size, 0, min(a.keep, first) - 1, a, qf, acc, m, l);
     warp_walk<T>(qs[warp], k_pages, v_pages, bt, p, h, hk, Hkv, dk, dv, page_size, first, p, a, qf, acc, m, l);
     T* orow = out + (size_t)t * out_stride + (size_t)h * dv;
     const float inv = a.out_scale / l;
 #pragma unroll
     for (int i = 0; i < NACC; ++i) {
         const int d = lane + 32 * i;
-        if (d < dv) orow[d] = from_f32<T>(acc[i] * inv);
+        if (d < dv) orow[d] = from_f32<T>(acc[i] * inv * gate_of<T>(a, t, h * dv + d));
     }
 }
 
@@ -193,7 +214,7 @@ attention_bias_split_kernel(const T* q, long long q_stride, const T* k_pages, co
     const bool live = wh < nh;
     const int seq = token_seq[t], p = positions[t];
     const int first = first_visible(a, p);
-    const int s_lo = max(first, split * SPLIT), s_hi = min(p, split * SPLIT + SPLIT - 1);
+    const int s_lo = split * SPLIT < a.keep ? split * SPLIT : max(first, split * SPLIT), s_hi = min(p, split * SPLIT + SPLIT - 1);
     if (s_lo > s_hi) {                                          // uniform over the CTA
         if (tid < nh) { const size_t pi = ((size_t)t * H + h0 + tid) * nsplit + split; part_ml[pi * 2] = -INFINITY; part_ml[pi * 2 + 1] = 0.f; }
         return;
@@ -215,6 +236,7 @@ attention_bias_split_kernel(const T* q, long long q_stride, const T* k_pages, co
     const int vpieces = (dv % VEC == 0 && ((uintptr_t)v_pages % 16) == 0) ? dv / VEC : 0;   // 0: value rows are copied by element
 
     for (int base = (s_lo / tile) * tile; base <= s_hi; base += tile) {
+        if (in_gap(a, base, base + tile - 1, first)) continue;  // uniform over the CTA
         __syncthreads();                                        // the tile before is no longer read; qs is complete
         constexpr int LD = 4;
         for (int i0 = tid; i0 < tile * kpieces; i0 += nthreads * LD) {
@@ -223,7 +245,7 @@ attention_bias_split_kernel(const T* q, long long q_stride, const T* k_pages, co
             for (int u = 0; u < LD; ++u) {
                 const int i = i0 + u * nthreads, key = i / kpieces, piece = i % kpieces, kp = base + key;
                 r[u] = make_uint4(0u, 0u, 0u, 0u);
-                if (i < tile * kpieces && kp >= s_lo && kp <= s_hi)
+                if (i < tile * kpieces && kp >= s_lo && kp <= s_hi && sees(a, kp, first))
                     r[u] = *reinterpret_cast<const uint4*>(k_pages + (((size_t)bt[kp / page_size] * Hkv + hk) * page_size + kp % page_size) * dk + piece * VEC);
             }
 #pragma unroll
@@ -239,7 +261,7 @@ attention_bias_split_kernel(const T* q, long long q_stride, const T* k_pages, co
                 for (int u = 0; u < LD; ++u) {
                     const int i = i0 + u * nthreads, key = i / vpieces, piece = i % vpieces, kp = base + key;
                     r[u] = make_uint4(0u, 0u, 0u, 0u);
-                    if (i < tile * vpieces && kp >= s_lo && kp <= s_hi)
+                    if (i < tile * vpieces && kp >= s_lo && kp <= s_hi && sees(a, kp, first))
                         r[u] = *reinterpret_cast<const uint4*>(v_pages + (((size_t)bt[kp / page_size] * Hkv + hk) * page_size + kp % page_size) * dv + piece * VEC);
                 }
 #pragma unroll
@@ -252,7 +274,7 @@ attention_bias_split_kernel(const T* q, long long q_stride, const T* k_pages, co
             for (int i = tid; i < tile * dv; i += nthreads) {
                 const int key = i / dv, d = i % dv, kp = base + key;
                 T val = from_f32<T>(0.f);
-                if (kp >= s_lo && kp <= s_hi)
+                if (kp >= s_lo && kp <= s_hi && sees(a, kp, first))
                     val = v_pages[(((size_t)bt[kp / page_size] * Hkv + hk) * page_size + kp % page_size) * dv + d];
                 Vs[(size_t)key * dv + d] = val;
             }
@@ -261,9 +283,9 @@ attention_bias_split_kernel(const T* q, long long q_stride, const T* k_pages, co
         for (int it = 0; it < NT; ++it) {
         const int ck = (it * KS + wk) * 32;                     // this warp's chunk of 32 keys within the tile
         const int c0 = base + ck;
-        if (!live || c0 > s_hi || c0 + 31 < s_lo) continue;     // uniform over the warp (barriers are outside)
+        if (!live || c0 > s_hi || c0 + 31 < s_lo || in_gap(a, c0, c0 + 31, first)) continue;     // uniform over the warp (barriers are outside)
         const int kp = c0 + lane;
-        const bool valid = kp >= s_lo && kp <= s_hi;
+        const bool valid = kp >= s_lo && kp <= s_hi && sees(a, kp, first);
         const T* kr = Ks + (size_t)(ck + lane) * krow;
         const float* qh = qs + wh * dk;
         float dot = 0.f;
@@ -339,13 +361,14 @@ template <typename T>
 __global__ void __launch_bounds__(WARPS * 32)
 attention_bias_merge_kernel(const float* part_o, const float* part_ml, const int* __restrict__ positions,
                             T* __restrict__ out, long long out_stride, int T_tokens, int H, int dv, int nsplit,
-                            float out_scale, const float* __restrict__ sink) {
+                            BiasArgs a) {
     pdl_wait();
     pdl_launch();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const long long gw = (long long)blockIdx.x * WARPS + warp;
     if (gw >= (long long)T_tokens * H) return;
     const int t = (int)(gw / H), h = (int)(gw % H);
+    const float* sink = a.sink;
     const int used = min(nsplit, positions[t] / SPLIT + 1);
     const size_t base = ((size_t)t * H + h) * nsplit;
     float mm = sink ? sink[h] : -INFINITY;
@@ -368,11 +391,11 @@ attention_bias_merge_kernel(const float* part_o, const float* part_ml, const int
         }
     }
     T* orow = out + (size_t)t * out_stride + (size_t)h * dv;
-    const float inv = out_scale / ll;
+    const float inv = a.out_scale / ll;
 #pragma unroll
     for (int i = 0; i < NACC; ++i) {
         const int d = lane + 32 * i;
-        if (d < dv) orow[d] = from_f32<T>(acc[i] * inv);
+        if (d < dv) orow[d] = from_f32<T>(acc[i] * inv * gate_of<T>(a, t, h * dv + d));
     }
 }
 
@@ -425,7 +448,8 @@ attention_bias_tiled_kernel(const T* q, long long q_stride, const T* k_pages, co
     const int q0 = pos0 + 2 * ty;           // absolute position of this thread's first row
     constexpr int VEC = 16 / sizeof(T);
 
-    for (int j = first_key / BK; j <= pos_max / BK; ++j) {
+    for (int j = a.keep > 0 ? 0 : first_key / BK; j <= pos_max / BK; ++j) {
+        if (in_gap(a, j * BK, j * BK + BK - 1, first_key)) continue;      // uniform over the CTA
         __syncthreads();                    // the previous tile is no longer read (and Qs is complete)
         const int kpieces = dk / VEC;
         for (int i = tid; i < BK * kpieces; i += THREADS) {
@@ -434,7 +458,7 @@ attention_bias_tiled_kernel(const T* q, long long q_stride, const T* k_pages, co
             float kf[8];
 #pragma unroll
             for (int e = 0; e < 8; ++e) kf[e] = 0.f;
-            if (kp <= pos_max && kp >= first_key) {
+            if (kp <= pos_max && sees(a, kp, first_key)) {
                 const int page = bt[kp / page_size];
                 const T* src = k_pages + (((size_t)page * Hkv + hk) * page_size + kp % page_size) * dk + piece * VEC;
                 if constexpr (sizeof(T) == 4) {
@@ -451,7 +475,7 @@ attention_bias_tiled_kernel(const T* q, long long q_stride, const T* k_pages, co
             const int key = i / dv, d = i % dv;
             const int kp = j * BK + key;
             float v = 0.f;
-            if (kp <= pos_max && kp >= first_key) {
+            if (kp <= pos_max && sees(a, kp, first_key)) {
                 const int page = bt[kp / page_size];
                 v = to_f32(v_pages[(((size_t)page * Hkv + hk) * page_size + kp % page_size) * dv + d]);
             }
@@ -486,7 +510,7 @@ attention_bias_tiled_kernel(const T* q, long long q_stride, const T* k_pages, co
 #pragma unroll
             for (int c = 0; c < 4; ++c) {
                 const int kp = j * BK + 4 * tx + c;
-                const bool vis = kp <= qp && qp <= pos_max && kp >= first_visible(a, qp);
+                const bool vis = kp <= qp && qp <= pos_max && sees(a, kp, first_visible(a, qp));
                 float sc = capped(s[r][c], a.softcap);
                 if (biased && vis) sc += Bs[qp - kp - dist0];
                 s[r][c] = vis ? sc : -INFINITY;
@@ -539,7 +563,8 @@ attention_bias_tiled_kernel(const T* q, long long q_stride, const T* k_pages, co
         T* orow = out + (size_t)(tok0 + row) * out_stride + (size_t)h * dv;
 #pragma unroll
         for (int i = 0; i < MAXI; ++i)
-            if (i < nd && tx + 8 * i < dv) orow[tx + 8 * i] = from_f32<T>(o[r][i] * inv);
+            if (i < nd && tx + 8 * i < dv)
+                orow[tx + 8 * i] = from_f32<T>(o[r][i] * inv * gate_of<T>(a, tok0 + row, h * dv + tx + 8 * i));
     }
 }
 
@@ -637,7 +662,7 @@ attention_bias_mma_kernel(const __nv_bfloat16* q, long long q_stride, const __nv
         for (int u = 0; u < SU; ++u) {
             if (k_kp[u] >= 0) {
                 const int key = k_kp[u] & 255, piece = k_kp[u] >> 8, kp = j * MK + key;
-                const bool ok = kp <= pos_max && kp >= first_key;
+                const bool ok = kp <= pos_max && sees(a, kp, first_key);
                 cp_async16(kd + key * krow + piece * 8, ok ? k_pages + row_of(kp) * dk + piece * 8 : k_pages, ok);
             }
         }
@@ -645,7 +670,7 @@ attention_bias_mma_kernel(const __nv_bfloat16* q, long long q_stride, const __nv
         for (int u = 0; u < SU; ++u) {
             if (v_kp[u] >= 0) {
                 const int key = v_kp[u] & 255, piece = v_kp[u] >> 8, kp = j * MK + key;
-                const bool ok = kp <= pos_max && kp >= first_key;
+                const bool ok = kp <= pos_max && sees(a, kp, first_key);
                 cp_async16(vd + key * vrow + piece * 8, ok ? v_pages + row_of(kp) * dv + piece * 8 : v_pages, ok);
             }
         }
@@ -661,7 +686,11 @@ attention_bias_mma_kernel(const __nv_bfloat16* q, long long q_stride, const __nv
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
 
-    const int j_first = first_key / MK, j_last = pos_max / MK;
+    const int j_first = a.keep > 0 ? 0 : first_key / MK, j_last = pos_max / MK;
+    auto after = [&](int j) {                                    // the next tile that some row of the CTA sees
+        ++j;
+        return in_gap(a, j * MK, j * MK + MK - 1, first_key) ? first_key / MK : j;
+    };
     for (int i = tid; i < MQ * kp8; i += 128) {                  // queries: rows beyond the tile are zero
         const int r = i / kp8, piece = i % kp8;
         cp_async16(Qs + r * qrow + piece * 8, r < rows ? q + (size_t)(tok0 + r) * q_stride + (size_t)h * dk + piece * 8 : q, r < rows);
@@ -685,11 +714,11 @@ attention_bias_mma_kernel(const __nv_bfloat16* q, long long q_stride, const __nv
     }
     const int nvt = dv / 8;
 
-    for (int j = j_first; j <= j_last; ++j) {
-        const int buf = (j - j_first) & 1;
+    for (int j = j_first, buf = 0, jn; j <= j_last; j = jn, buf ^= 1) {
+        jn = after(j);
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();                                         // tile j is in; the other buffer is free
-        if (j < j_last) stage(j + 1, buf ^ 1);
+        if (jn <= j_last) stage(jn, buf ^ 1);
         const bf* kt = Ks + buf * MK * krow;
         const bf* vt = Vs + buf * MK * vrow;
         const float* bs = Bs + buf * (MQ + MK);
@@ -711,8 +740,9 @@ attention_bias_mma_kernel(const __nv_bfloat16* q, long long q_stride, const __nv
         // log2 e), so that the exponentials are exp2.  A tile that every row of the warp sees whole needs no mask.
         const int dist0 = pos0 - (j * MK + MK - 1);
         const int w_lo = pos0 + warp * 16, w_hi = w_lo + 15;
-        const bool whole = j * MK + MK - 1 <= w_lo && w_hi <= pos_max && (a.window <= 0 || j * MK > w_hi - a.window) &&
-                           (a.chunk <= 0 || j * MK >= (w_hi / a.chunk) * a.chunk);
+        const bool whole = j * MK + MK - 1 <= w_lo && w_hi <= pos_max &&
+                           (((a.window <= 0 || j * MK > w_hi - a.window) && (a.chunk <= 0 || j * MK >= (w_hi / a.chunk) * a.chunk)) ||
+                            j * MK + MK <= a.keep);
         float mx0 = -INFINITY, mx1 = -INFINITY;
         if (whole) {
             const float* b0 = bs + (qp0 - j * MK - dist0) - 2 * (lane & 3);      // bias of (row r0, key j*MK + 2*(lane&3)); keys go down
@@ -734,7 +764,7 @@ attention_bias_mma_kernel(const __nv_bfloat16* q, long long q_stride, const __nv
                 for (int e = 0; e < 4; ++e) {
                     const int kp = j * MK + n * 8 + 2 * (lane & 3) + (e & 1);
                     const int qp = (e < 2) ? qp0 : qp1;
-                    const bool vis = kp <= qp && qp <= pos_max && kp >= first_visible(a, qp);
+                    const bool vis = kp <= qp && qp <= pos_max && sees(a, kp, first_visible(a, qp));
                     float sc = s[n][e] * ((e < 2) ? qf0 : qf1);
                     if (a.softcap > 0.f) sc = capl * tanhf(sc);
                     if (biased && vis) sc += bs[qp - kp - dist0];
@@ -795,12 +825,16 @@ attention_bias_mma_kernel(const __nv_bfloat16* q, long long q_stride, const __nv
     for (int i = 0; i < NO; ++i) {
         if (i < nvt) {
             const int col = i * 8 + 2 * (lane & 3);
-            if (r0 < rows)
-                *reinterpret_cast<__nv_bfloat162*>(out + (size_t)(tok0 + r0) * out_stride + (size_t)h * dv + col) =
-                    __floats2bfloat162_rn(o[i][0] * inv0, o[i][1] * inv0);
-            if (r0 + 8 < rows)
-                *reinterpret_cast<__nv_bfloat162*>(out + (size_t)(tok0 + r0 + 8) * out_stride + (size_t)h * dv + col) =
-                    __floats2bfloat162_rn(o[i][2] * inv1, o[i][3] * inv1);
+            if (r0 < rows) {
+                const int t = tok0 + r0, gc = h * dv + col;
+                *reinterpret_cast<__nv_bfloat162*>(out + (size_t)t * out_stride + gc) =
+                    __floats2bfloat162_rn(o[i][0] * inv0 * gate_of<bf>(a, t, gc), o[i][1] * inv0 * gate_of<bf>(a, t, gc + 1));
+            }
+            if (r0 + 8 < rows) {
+                const int t = tok0 + r0 + 8, gc = h * dv + col;
+                *reinterpret_cast<__nv_bfloat162*>(out + (size_t)t * out_stride + gc) =
+                    __floats2bfloat162_rn(o[i][2] * inv1 * gate_of<bf>(a, t, gc), o[i][3] * inv1 * gate_of<bf>(a, t, gc + 1));
+            }
         }
     }
 }
@@ -829,13 +863,15 @@ MLLM_EXPORT int mllm_attention_bias(const void* q, long long q_stride, const voi
                                     float* part_ml, int nsplit, int T, int H, int Hkv, int dkq, int dk, int dv, int page_size,
                                     float scale, float out_scale, const float* dist_bias, int n_dist,
                                     const float* q_scale, int window, int chunk, const float* sink, float softcap,
-                                    const float* slopes, int dtype, int impl, cudaStream_t stream) {
+                                    const float* slopes, int keep_first, const void* gate, long long gate_stride, int dtype, int impl,
+                                    cudaStream_t stream) {
     if (T <= 0) return 0;
     if (int rc = check_sizes(H, Hkv, dk, dv, page_size, dtype)) return rc;
     if (dkq <= 0 || dkq > dk) return mllm_fail(1, "attention_bias: queries of %d against key rows of %d", dkq, dk);
     if (window < 0 || chunk < 0) return mllm_fail(1, "attention_bias: window %d, chunk %d", window, chunk);
+    if (keep_first < 0) return mllm_fail(1, "attention_bias: %d kept keys", keep_first);
     if (!(softcap >= 0.f)) return mllm_fail(1, "attention_bias: a cap of %g on the scores", (double)softcap);
-    BiasArgs a{dist_bias, n_dist, q_scale, scale, out_scale, window, chunk, sink, softcap, slopes};
+    BiasArgs a{dist_bias, n_dist, q_scale, scale, out_scale, window, chunk, sink, softcap, slopes, keep_first, gate, gate_stride};
     const long long warps = (long long)T * H;
     const long long blocks = (warps + WARPS - 1) / WARPS;
     if (blocks > 2147483647LL) return mllm_fail(1, "attention_bias: too many (token, head) pairs");
@@ -903,7 +939,7 @@ MLLM_EXPORT int mllm_attention_bias(const void* q, long long q_stride, const voi
                                   bt_stride, token_seq, positions, part_o, part_ml, H, Hkv, dkq, dk, dv, page_size, HG, KS, NT, a));
             MLLM_CUDA(mllm_launch(attention_bias_merge_kernel<float>, dim3((unsigned)blocks), dim3(WARPS * 32), 0, stream, true,
                                   (const float*)part_o, (const float*)part_ml, positions, (float*)out, out_stride, T, H, dv,
-                                  nsplit, out_scale, a.sink));
+                                  nsplit, a));
         } else {
             if (smem > 48 * 1024) MLLM_CUDA(cudaFuncSetAttribute(attention_bias_split_kernel<bf>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
             MLLM_CUDA(mllm_launch(attention_bias_split_kernel<bf>, grid, block, smem, stream, true,
@@ -911,7 +947,7 @@ MLLM_EXPORT int mllm_attention_bias(const void* q, long long q_stride, const voi
                                   token_seq, positions, part_o, part_ml, H, Hkv, dkq, dk, dv, page_size, HG, KS, NT, a));
             MLLM_CUDA(mllm_launch(attention_bias_merge_kernel<bf>, dim3((unsigned)blocks), dim3(WARPS * 32), 0, stream, true,
                                   (const float*)part_o, (const float*)part_ml, positions, (bf*)out, out_stride, T, H, dv,
-                                  nsplit, out_scale, a.sink));
+                                  nsplit, a));
         }
         return 0;
     }

@@ -1,6 +1,6 @@
 // Token embedding gather with the additive position table fused in:
-// x[t,:] = table[id_t,:] * scale (+ pos_table[pos_t,:]), written as 32-bit, and once more to `keep` when a later part of the
-// model reads the embedded rows again.
+// x[t,:] = table[id_t,:] * scale (+ pos_table[pos_t,:]), written as 32-bit, once more to `keep` when a later part of the
+// model reads the embedded rows again, and to `act` in the table's dtype when the first layer's products read x itself.
 // Same arithmetic as the reference's embedding_kernel (src/kernels/embedding.cu:23-43),
 // for any width and either table dtype; row offsets are 64-bit.
 #include "common.cuh"
@@ -8,7 +8,7 @@
 template <typename T>
 __global__ void embed_kernel(const int* __restrict__ ids, const int* __restrict__ pos,
                              const T* __restrict__ table, const T* __restrict__ pos_table,
-                             float* __restrict__ out, float* __restrict__ keep, int D, int copies, float scale) {
+                             float* __restrict__ out, float* __restrict__ keep, T* __restrict__ act, int D, int copies, float scale) {
     const int t = blockIdx.x;
     pdl_launch();               // the first kernel of a step: nothing before it to wait for
     const T* row = table + (size_t)ids[t] * D;
@@ -18,21 +18,22 @@ __global__ void embed_kernel(const int* __restrict__ ids, const int* __restrict_
         float v = to_f32(row[d]) * scale;
         if (prow) v += to_f32(prow[d]);
         if (keep) keep[(size_t)t * D + d] = v;
+        if (act) act[(size_t)t * D + d] = from_f32<T>(v);
         for (int c = 0; c < copies; ++c) o[(size_t)c * D + d] = v;     // a residual of several streams starts as copies
     }
 }
 
 MLLM_EXPORT int mllm_embed(const int* ids, const int* pos, const void* table, const void* pos_table,
-                           float* out, float* keep, int T, int D, int copies, float scale, int dtype, cudaStream_t stream) {
+                           float* out, float* keep, void* act, int T, int D, int copies, float scale, int dtype, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (D <= 0 || copies <= 0) return mllm_fail(1, "embed: width %d, %d copies", D, copies);
     int threads = D >= 256 ? 256 : ((D + 31) / 32) * 32;
     if (dtype == MLLM_F32)
-        embed_kernel<float><<<T, threads, 0, stream>>>(ids, pos, (const float*)table, (const float*)pos_table, out, keep, D, copies,
+        embed_kernel<float><<<T, threads, 0, stream>>>(ids, pos, (const float*)table, (const float*)pos_table, out, keep, (float*)act, D, copies,
                                                     scale);
     else if (dtype == MLLM_BF16)
         embed_kernel<__nv_bfloat16><<<T, threads, 0, stream>>>(ids, pos, (const __nv_bfloat16*)table,
-                                                               (const __nv_bfloat16*)pos_table, out, keep, D, copies, scale);
+                                                               (const __nv_bfloat16*)pos_table, out, keep, (__nv_bfloat16*)act, D, copies, scale);
     else
         return mllm_fail(1, "embed: unknown dtype code %d", dtype);
     MLLM_CHECK_LAUNCH("embed");
@@ -92,5 +93,37 @@ MLLM_EXPORT int mllm_concat_terms(const float* x, long long x_stride, const floa
                               x0_stride, (__nv_bfloat16*)out, out_stride, D));
     else
         return mllm_fail(1, "concat_terms: %d terms of dtype code %d", terms, dtype);
+    return 0;
+}
+
+// A per-layer input of the token: out[t][c] = gelu_tanh(z[t][c]) * table[ids[t]][off + c], c < d; z 32-bit, table and out in
+// the activation dtype.
+template <typename T>
+__global__ void __launch_bounds__(256)
+token_side_gate_kernel(const float* z, long long ldz, const int* __restrict__ ids, const T* __restrict__ table, long long ldt, int off,
+                       T* __restrict__ out, long long ldo, int rows, int d) {
+    pdl_wait();
+    pdl_launch();
+    const long long total = (long long)rows * d;
+    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+        const int t = (int)(i / d), c = (int)(i % d);
+        out[(size_t)t * ldo + c] = from_f32<T>(gelu_tanh_f(z[(size_t)t * ldz + c]) * to_f32(table[(size_t)ids[t] * ldt + off + c]));
+    }
+}
+
+MLLM_EXPORT int mllm_token_side_gate(const float* z, long long ldz, const int* ids, const void* table, long long ldt, int off, void* out,
+                                     long long ldo, int T, int d, int dtype, cudaStream_t stream) {
+    if (T <= 0) return 0;
+    if (d <= 0 || off < 0 || off + d > ldt) return mllm_fail(1, "token_side_gate: columns %d to %d of rows of %lld", off, off + d, ldt);
+    const long long total = (long long)T * d;
+    const int grid = (int)((total + 255) / 256 < 8192 ? (total + 255) / 256 : 8192);
+    if (dtype == MLLM_F32)
+        MLLM_CUDA(mllm_launch(token_side_gate_kernel<float>, dim3(grid), dim3(256), 0, stream, true, z, ldz, ids, (const float*)table, ldt,
+                              off, (float*)out, ldo, T, d));
+    else if (dtype == MLLM_BF16)
+        MLLM_CUDA(mllm_launch(token_side_gate_kernel<__nv_bfloat16>, dim3(grid), dim3(256), 0, stream, true, z, ldz, ids,
+                              (const __nv_bfloat16*)table, ldt, off, (__nv_bfloat16*)out, ldo, T, d));
+    else
+        return mllm_fail(1, "token_side_gate: unknown dtype code %d", dtype);
     return 0;
 }

@@ -7,6 +7,8 @@
 //                   experts: the `top` largest logits are chosen and the weights are the softmax over those alone.
 //                   `mode` 2: the scores are sigmoid(logit), each expert's on its own.  `group_sum` 2: a group's score is
 //                   the sum of its two largest scores instead of its largest.  The weights are multiplied by `w_scale`.
+//                   `correction` (no groups): a number per expert is added to the scores for the choice alone.  `renorm` 0:
+//                   the weights are the chosen scores as they are.  `Wg`: one more row; sigmoid(Wg x) goes to gate[t].
 //   moe_sort        one CTA: the (token, choice) pairs ordered by expert (a counting sort) and the experts' offsets;
 //                   with up to 16 tokens (decode steps) routing and ordering are one launch of one CTA.
 //   moe_grouped     out[row] = A[a_row] W_e^T for the pairs of expert e; a CTA finds its expert from the offsets on the
@@ -15,6 +17,8 @@
 //                   gate has W_e [F, K] and an activation of one argument on the product (`uact`: the square of relu).  Three kernels: CUDA cores, 32 pairs x 64 columns per
 //                   CTA (32-bit weights, odd sizes); tensor cores, 64 x 64 (bfloat16); and for up to 32 pairs (decode
 //                   steps) a CTA per pair and 64 columns whose warps stream the weight rows.
+//                   Identity experts (numbers E .. E_total - 1, no weights): their pairs stand last in the order; the first
+//                   product leaves them out and the second copies the token's input row to the pair's result.
 //   moe_combine     y[t] (+)= sum_k weight[t][k] * pair_out[t * top + k], in the order of k.
 // A row of a product depends on that row's input only, so a token's result does not depend on what else is in the batch.
 #include "common.cuh"
@@ -25,11 +29,45 @@ constexpr int MAX_E = 512;
 constexpr int MOE_FEW_TOKENS = 16;    // up to this many tokens one CTA routes them all and orders the pairs in the same launch
 constexpr int MOE_FEW_PAIRS = 32;     // up to this many (token, choice) pairs every pair streams its expert's weights itself
 
+template <typename T>
+struct RouteArgs {
+    const T* Wr;                    // [E][D]
+    const float* bias;              // [E] or null: on the logits
+    const float* correction;        // [E] or null: on the scores, for the choice alone
+    const T* Wg;                    // [D] or null: a gate per token
+    float* gate;                    // [T]
+    int mode, D, E, top, n_groups, keep, group_sum, renorm;
+    float w_scale;
+};
+
+// sigmoid(Wg x) of one token by one warp
+template <typename T>
+__device__ __forceinline__ void token_gate(const T* x, const T* __restrict__ Wg, int D, float* gate, int lane) {
+    constexpr int V = 16 / sizeof(T);
+    float acc = 0.f;
+    if (D % V == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)Wg % 16 == 0) {
+        for (int d = lane * V; d < D; d += 32 * V) {
+            const uint4 xv = *reinterpret_cast<const uint4*>(x + d), wv = *reinterpret_cast<const uint4*>(Wg + d);
+            const T* px = reinterpret_cast<const T*>(&xv);
+            const T* pw = reinterpret_cast<const T*>(&wv);
+#pragma unroll
+            for (int c = 0; c < V; ++c) acc = fmaf(to_f32(px[c]), to_f32(pw[c]), acc);
+        }
+    } else {
+        for (int d = lane; d < D; d += 32) acc = fmaf(to_f32(x[d]), to_f32(Wg[d]), acc);
+    }
+    acc = warp_sum(acc);
+    if (lane == 0) *gate = 1.0f / (1.0f + expf(-acc));
+}
+
 // One warp routes one token; `s` is the warp's E floats of shared memory.
 template <typename T>
-__device__ __forceinline__ void route_token(const T* x, const T* __restrict__ Wr, const float* __restrict__ bias, int mode,
-                                            float* s, int D, int E, int top, int n_groups, int keep, int group_sum,
-                                            float w_scale, int* idx, float* wout, int lane) {
+__device__ __forceinline__ void route_token(const T* x, const RouteArgs<T>& ra, float* s, int* idx, float* wout, int t, int lane) {
+    const T* __restrict__ Wr = ra.Wr;
+    const float* __restrict__ bias = ra.bias;
+    const int mode = ra.mode, D = ra.D, E = ra.E, top = ra.top, n_groups = ra.n_groups, keep = ra.keep, group_sum = ra.group_sum;
+    const float w_scale = ra.w_scale;
+    if (ra.Wg) token_gate(x, ra.Wg, D, ra.gate + t, lane);
     constexpr int V = 16 / sizeof(T);                           // elements per 16-byte load
     const bool vec = D % V == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)Wr % 16 == 0;
     for (int e0 = 0; e0 < E; e0 += 4) {                         // four experts at a time: their loads are in flight together
@@ -112,6 +150,37 @@ __device__ __forceinline__ void route_token(const T* x, const T* __restrict__ Wr
         for (int e = lane; e < E; e += 32) s[e] = s[e] / sum;
     }
     __syncwarp();
+    if (n_groups == 1) {
+        // the warp looks for the largest together: a lane's experts are lane, lane + 32, ..., and among equals the lowest wins
+        float wsum = 0.f;
+        for (int k = 0; k < top; ++k) {
+            int best = E;
+            float bv = -INFINITY;
+            for (int e = lane; e < E; e += 32) {
+                const float v = ra.correction ? s[e] + ra.correction[e] : s[e];
+                if (s[e] >= 0.f && (best == E || v > bv)) { bv = v; best = e; }
+            }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) {
+                const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
+                const int ob = __shfl_xor_sync(0xffffffffu, best, o);
+                if (ob < E && (best == E || ov > bv || (ov == bv && ob < best))) { bv = ov; best = ob; }
+            }
+            best = min(best, E - 1);                             // never beyond the experts, whatever the scores are
+            const float sc = s[best];
+            __syncwarp();
+            if (lane == 0) {
+                idx[k] = best;
+                wout[k] = sc;
+                s[best] = -1.f;                                  // taken (scores are >= 0)
+            }
+            wsum += sc;
+            __syncwarp();
+        }
+        for (int k = lane; k < top; k += 32) wout[k] = ra.renorm ? wout[k] / (wsum + 1e-20f) * w_scale : wout[k] * w_scale;
+        __syncwarp();
+        return;
+    }
     if (lane == 0) {
         // experts outside the kept groups are marked by a negative score (scores are >= 0)
         if (n_groups > 1 && keep < n_groups) {
@@ -147,7 +216,7 @@ __device__ __forceinline__ void route_token(const T* x, const T* __restrict__ Wr
             wsum += bv;
             s[best] = -8.f;                                  // taken
         }
-        for (int k = 0; k < top; ++k) wout[k] = wout[k] / (wsum + 1e-20f) * w_scale;
+        for (int k = 0; k < top; ++k) wout[k] = ra.renorm ? wout[k] / (wsum + 1e-20f) * w_scale : wout[k] * w_scale;
     }
     __syncwarp();
 }
@@ -187,15 +256,13 @@ __device__ __forceinline__ void sort_pairs(const int* idx, int n, int E, int* of
 // 4 warps, a token each; dynamic shared memory: 4 * E floats
 template <typename T>
 __global__ void __launch_bounds__(128)
-moe_route_kernel(const T* h, long long ld, const T* __restrict__ Wr, const float* __restrict__ bias, int mode, int Tn, int D,
-                 int E, int top, int n_groups, int keep, int group_sum, float w_scale, int* idx, float* wout) {
+moe_route_kernel(const T* h, long long ld, int Tn, int* idx, float* wout, RouteArgs<T> ra) {
     extern __shared__ float sc[];
     pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x * 4 + warp;
     if (t >= Tn) return;
-    route_token(h + (size_t)t * ld, Wr, bias, mode, sc + warp * E, D, E, top, n_groups, keep, group_sum, w_scale,
-                idx + (size_t)t * top, wout + (size_t)t * top, lane);
+    route_token(h + (size_t)t * ld, ra, sc + warp * ra.E, idx + (size_t)t * ra.top, wout + (size_t)t * ra.top, t, lane);
 }
 
 __global__ void __launch_bounds__(1024)
@@ -209,16 +276,14 @@ moe_sort_kernel(const int* idx, int n, int E, int* offsets, int* sorted) {
 // dynamic shared memory: 8 * E floats, then E + 1 ints
 template <typename T>
 __global__ void __launch_bounds__(256)
-moe_route_sort_kernel(const T* h, long long ld, const T* __restrict__ Wr, const float* __restrict__ bias, int mode, int Tn,
-                      int D, int E, int top, int n_groups, int keep, int group_sum, float w_scale, int* idx, float* wout,
-                      int* offsets, int* sorted) {
+moe_route_sort_kernel(const T* h, long long ld, int Tn, int* idx, float* wout, int* offsets, int* sorted, RouteArgs<T> ra) {
     extern __shared__ float sc[];
+    const int E = ra.E, top = ra.top;
     int* cnt = reinterpret_cast<int*>(sc + 8 * E);
     pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     for (int t = warp; t < Tn; t += 8)
-        route_token(h + (size_t)t * ld, Wr, bias, mode, sc + warp * E, D, E, top, n_groups, keep, group_sum, w_scale,
-                    idx + (size_t)t * top, wout + (size_t)t * top, lane);
+        route_token(h + (size_t)t * ld, ra, sc + warp * E, idx + (size_t)t * top, wout + (size_t)t * top, t, lane);
     __syncthreads();                                         // the CTA's own writes of idx are visible to all its threads
     sort_pairs(idx, Tn * top, E, offsets, sorted, cnt);
 }
@@ -231,11 +296,19 @@ __device__ __forceinline__ float unary_act(float v, int uact) {
     return v;
 }
 
+// the input rows that identity experts give back (second product only): rows null means none
+template <typename TA>
+struct SelfRows {
+    const TA* rows;
+    long long ld;
+    int E_total, top;
+};
+
 template <typename TA, typename TW, typename TO>
 __global__ void __launch_bounds__(256)
 moe_grouped_kernel(const TA* A, long long lda, const TW* __restrict__ W, TO* out, long long ldo, const int* offsets,
                    const int* sorted, int E, int N, int K, int a_div, int out_by_pair, int gated, float limit, float alpha,
-                   int uact) {
+                   int uact, SelfRows<TA> self) {
     __shared__ float As[32][33];
     __shared__ float Ws[64][33];
     __shared__ float Us[64][33];
@@ -250,6 +323,10 @@ moe_grouped_kernel(const TA* A, long long lda, const TW* __restrict__ W, TO* out
             if (tile < tiles) { found = e; r0 = lo + tile * 32; c = min(32, n - tile * 32); break; }
             tile -= tiles;
         }
+        if (found < 0 && self.rows) {
+            const int lo = offsets[E] + tile * 32, n = offsets[self.E_total] - lo;
+            if (n > 0) { found = E; r0 = lo; c = min(32, n); }
+        }
         s_e = found; s_r0 = r0; s_cnt = c;
     }
     __syncthreads();
@@ -263,6 +340,13 @@ moe_grouped_kernel(const TA* A, long long lda, const TW* __restrict__ W, TO* out
     }
     __syncthreads();
     const int n0 = blockIdx.y * 64;
+    if (e >= E) {                                               // identity experts: the token's own row
+        for (int i = threadIdx.x; i < cnt * 64; i += 256) {
+            const int r = i >> 6, col = n0 + (i & 63);
+            if (col < N) out[(size_t)rows_o[r] * ldo + col] = from_f32<TO>(to_f32(self.rows[(size_t)(rows_o[r] / self.top) * self.ld + col]));
+        }
+        return;
+    }
     const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
     const size_t wrows = gated ? (size_t)2 * N : (size_t)N;
     const TW* We = W + (size_t)e * wrows * K;
@@ -323,11 +407,19 @@ template <typename TA, typename TW, typename TO>
 __global__ void __launch_bounds__(256)
 moe_rows_kernel(const TA* A, long long lda, const TW* __restrict__ W, TO* out, long long ldo, const int* offsets,
                 const int* sorted, int E, int N, int K, int a_div, int out_by_pair, int gated, float limit, float alpha,
-                int uact) {
+                int uact, SelfRows<TA> self) {
     extern __shared__ float xs[];                                // [K]
     __shared__ int s_e;
     pdl_wait();
     const int i = blockIdx.x;
+    if (i >= offsets[E]) {                                       // a pair of an identity expert (uniform over the CTA)
+        const int col = blockIdx.y * 64 + threadIdx.x;
+        if (self.rows && threadIdx.x < 64 && col < N) {
+            const int p = sorted[i];
+            out[(size_t)(out_by_pair ? p : i) * ldo + col] = from_f32<TO>(to_f32(self.rows[(size_t)(p / self.top) * self.ld + col]));
+        }
+        return;
+    }
     if (threadIdx.x == 0) {
         int e = 0;
         while (e < E - 1 && offsets[e + 1] <= i) ++e;
@@ -415,7 +507,7 @@ template <typename TO, int GATED>
 __global__ void __launch_bounds__(128)
 moe_grouped_mma_kernel(const __nv_bfloat16* A, long long lda, const __nv_bfloat16* __restrict__ W, TO* out, long long ldo,
                        const int* offsets, const int* sorted, int E, int N, int K, int a_div, int out_by_pair, int act,
-                       float limit, float alpha) {
+                       float limit, float alpha, SelfRows<__nv_bfloat16> self) {
     using bf = __nv_bfloat16;
     extern __shared__ __align__(16) unsigned char gsm[];
     constexpr int STAGE = (GM + GN * (1 + GATED)) * GROW;        // elements per stage
@@ -432,6 +524,10 @@ moe_grouped_mma_kernel(const __nv_bfloat16* A, long long lda, const __nv_bfloat1
             if (tile < tiles) { found = e; r0 = lo + tile * GM; c = min(GM, n - tile * GM); break; }
             tile -= tiles;
         }
+        if (found < 0 && self.rows) {
+            const int lo = offsets[E] + tile * GM, n = offsets[self.E_total] - lo;
+            if (n > 0) { found = E; r0 = lo; c = min(GM, n); }
+        }
         s_e = found; s_r0 = r0; s_cnt = c;
     }
     __syncthreads();
@@ -445,6 +541,13 @@ moe_grouped_mma_kernel(const __nv_bfloat16* A, long long lda, const __nv_bfloat1
     }
     __syncthreads();
     const int n0 = blockIdx.y * GN;
+    if (e >= E) {                                               // identity experts: the token's own row
+        for (int i = tid; i < cnt * GN; i += 128) {
+            const int r = i / GN, col = n0 + i % GN;
+            if (col < N) out[(size_t)rows_o[r] * ldo + col] = from_f32<TO>(to_f32(self.rows[(size_t)(rows_o[r] / self.top) * self.ld + col]));
+        }
+        return;
+    }
     const bf* We = W + (size_t)e * (size_t)(1 + GATED) * N * K;
     auto stage = [&](int k0, int buf) {
         bf* As = sm + buf * STAGE;
@@ -524,40 +627,41 @@ moe_combine_kernel(const float* pair_out, const float* w, float* y, long long ld
 
 MLLM_EXPORT int mllm_moe_max_experts() { return MAX_E; }
 
+// correction [E] or null; Wg [D] with gate [Tn], or null.
 MLLM_EXPORT int mllm_moe_route(const void* h, long long ld, const void* Wr, const float* bias, int mode, int Tn, int D, int E,
-                               int top, int n_groups, int keep, int group_sum, float w_scale, int* idx, float* w, int* offsets,
-                               int* sorted, int dtype, cudaStream_t stream) {
+                               int top, int n_groups, int keep, int group_sum, float w_scale, const float* correction, int renorm,
+                               const void* Wg, float* gate, int* idx, float* w, int* offsets, int* sorted, int dtype,
+                               cudaStream_t stream) {
     if (Tn <= 0) return 0;
     if (mode < 0 || mode > 2) return mllm_fail(1, "moe_route: unknown mode %d", mode);
     if (group_sum != 1 && group_sum != 2) return mllm_fail(1, "moe_route: a group's score is its largest score or the sum of its two largest, not of %d", group_sum);
+    if (correction && (mode == 1 || n_groups != 1)) return mllm_fail(1, "moe_route: a correction of the choice takes scores over all experts and no groups");
+    if (mode == 1 && !renorm) return mllm_fail(1, "moe_route: the softmax over the chosen logits has no other weights");
+    if (Wg && !gate) return mllm_fail(1, "moe_route: a gate per token without a place for it");
     if (mode == 1 && n_groups != 1) return mllm_fail(1, "moe_route: the softmax over the chosen logits takes no groups");
     if (E < 1 || E > MAX_E || top < 1 || top > E) return mllm_fail(1, "moe_route: %d experts (at most %d), top %d", E, MAX_E, top);
     if (n_groups < 1 || E % n_groups || keep < 1 || keep > n_groups || n_groups > 64)
         return mllm_fail(1, "moe_route: %d experts in %d groups (at most 64), %d kept", E, n_groups, keep);
     if (keep * (E / n_groups) < top) return mllm_fail(1, "moe_route: %d kept groups of %d experts cannot give %d", keep, E / n_groups, top);
+    using bf = __nv_bfloat16;
+    if (dtype != MLLM_F32 && dtype != MLLM_BF16) return mllm_fail(1, "moe_route: unknown dtype code %d", dtype);
+    const RouteArgs<float> rf{(const float*)Wr, bias, correction, (const float*)Wg, gate, mode, D, E, top, n_groups, keep, group_sum, renorm, w_scale};
+    const RouteArgs<bf> rb{(const bf*)Wr, bias, correction, (const bf*)Wg, gate, mode, D, E, top, n_groups, keep, group_sum, renorm, w_scale};
     if (Tn <= MOE_FEW_TOKENS) {
         const size_t smem = (size_t)8 * E * 4 + (size_t)(E + 1) * 4;
         if (dtype == MLLM_F32)
-            MLLM_CUDA(mllm_launch(moe_route_sort_kernel<float>, dim3(1), dim3(256), smem, stream, true, (const float*)h, ld,
-                                  (const float*)Wr, bias, mode, Tn, D, E, top, n_groups, keep, group_sum, w_scale, idx, w, offsets, sorted));
-        else if (dtype == MLLM_BF16)
-            MLLM_CUDA(mllm_launch(moe_route_sort_kernel<__nv_bfloat16>, dim3(1), dim3(256), smem, stream, true,
-                                  (const __nv_bfloat16*)h, ld, (const __nv_bfloat16*)Wr, bias, mode, Tn, D, E, top, n_groups, keep,
-                                  group_sum, w_scale, idx, w, offsets, sorted));
+            MLLM_CUDA(mllm_launch(moe_route_sort_kernel<float>, dim3(1), dim3(256), smem, stream, true, (const float*)h, ld, Tn, idx, w,
+                                  offsets, sorted, rf));
         else
-            return mllm_fail(1, "moe_route: unknown dtype code %d", dtype);
+            MLLM_CUDA(mllm_launch(moe_route_sort_kernel<bf>, dim3(1), dim3(256), smem, stream, true, (const bf*)h, ld, Tn, idx, w,
+                                  offsets, sorted, rb));
         return 0;
     }
     const size_t smem = (size_t)4 * E * 4;
     if (dtype == MLLM_F32)
-        MLLM_CUDA(mllm_launch(moe_route_kernel<float>, dim3((Tn + 3) / 4), dim3(128), smem, stream, true, (const float*)h, ld,
-                              (const float*)Wr, bias, mode, Tn, D, E, top, n_groups, keep, group_sum, w_scale, idx, w));
-    else if (dtype == MLLM_BF16)
-        MLLM_CUDA(mllm_launch(moe_route_kernel<__nv_bfloat16>, dim3((Tn + 3) / 4), dim3(128), smem, stream, true,
-                              (const __nv_bfloat16*)h, ld, (const __nv_bfloat16*)Wr, bias, mode, Tn, D, E, top, n_groups, keep,
-                              group_sum, w_scale, idx, w));
+        MLLM_CUDA(mllm_launch(moe_route_kernel<float>, dim3((Tn + 3) / 4), dim3(128), smem, stream, true, (const float*)h, ld, Tn, idx, w, rf));
     else
-        return mllm_fail(1, "moe_route: unknown dtype code %d", dtype);
+        MLLM_CUDA(mllm_launch(moe_route_kernel<bf>, dim3((Tn + 3) / 4), dim3(128), smem, stream, true, (const bf*)h, ld, Tn, idx, w, rb));
     MLLM_CUDA(mllm_launch(moe_sort_kernel, dim3(1), dim3(1024), 0, stream, true, (const int*)idx, Tn * top, E, offsets, sorted));
     return 0;
 }
@@ -569,11 +673,19 @@ MLLM_EXPORT int mllm_moe_few_tokens() { return MOE_FEW_TOKENS; }
 // kind 1: A in `dtype`, out 32-bit (the experts' second product);
 // kind 2: A in `dtype`, no gate, out in `dtype` = act(A W_e^T) with an activation of one argument (MLLM_ACT_RELU_SQ ...):
 // the first product of experts without a gate.
+// Experts E .. E_total - 1 are identity experts: kinds 0 and 2 leave their pairs out; kind 1 copies the rows of `self` (the
+// tokens' inputs in `dtype`, row = pair / self_top).  The offsets hold E_total + 1 entries.
 MLLM_EXPORT int mllm_moe_grouped(const void* A, long long lda, const void* W, void* out, long long ldo, const int* offsets,
                                  const int* sorted, int n_pairs, int E, int N, int K, int a_div, int out_by_pair, int kind,
-                                 int act, float limit, float alpha, int dtype, cudaStream_t stream) {
+                                 int act, float limit, float alpha, const void* self, long long ldself, int E_total, int self_top,
+                                 int dtype, cudaStream_t stream) {
     if (n_pairs <= 0 || N <= 0) return 0;
-    const dim3 grid((n_pairs + 31) / 32 + E, (N + 63) / 64), block(256);
+    if (E_total < E || (self && (kind != 1 || self_top < 1)) || (kind == 1 && E_total > E && !self))
+        return mllm_fail(1, "moe_grouped: %d of %d experts with weights, kind %d", E, E_total, kind);
+    const SelfRows<float> sf{(const float*)self, ldself, E_total, self_top};
+    const SelfRows<__nv_bfloat16> sb{(const __nv_bfloat16*)self, ldself, E_total, self_top};
+    const int id_tile = E_total > E ? 1 : 0;                     // the identity pairs' last, partly filled tile
+    const dim3 grid((n_pairs + 31) / 32 + E + id_tile, (N + 63) / 64), block(256);
     if (grid.y > 65535) return mllm_fail(1, "moe_grouped: too many columns");
     if (kind == 0 && act != MLLM_ACT_SILU && act != MLLM_ACT_SWIGLU_CLAMP) return mllm_fail(1, "moe_grouped: activation code %d", act);
     if (kind == 2 && act != MLLM_ACT_RELU_SQ && act != MLLM_ACT_RELU && act != MLLM_ACT_GELU_TANH)
@@ -584,7 +696,7 @@ MLLM_EXPORT int mllm_moe_grouped(const void* A, long long lda, const void* W, vo
     if (n_pairs <= MOE_FEW_PAIRS && (size_t)K * 4 <= 96 * 1024) {
         const dim3 fg(n_pairs, (N + 63) / 64);
         const size_t smem = (size_t)K * 4;
-#define MLLM_ROWS(TA, TW, TO)                                                                                            \
+#define MLLM_ROWS(TA, TW, TO, SELF)                                                                                            \
         do {                                                                                                             \
             static bool raised = false;                                                                                  \
             if (smem > 48 * 1024 && !raised) {                                                                           \
@@ -592,17 +704,17 @@ MLLM_EXPORT int mllm_moe_grouped(const void* A, long long lda, const void* W, vo
                 raised = true;                                                                                           \
             }                                                                                                            \
             MLLM_CUDA(mllm_launch(moe_rows_kernel<TA, TW, TO>, fg, block, smem, stream, true, (const TA*)A, lda, (const TW*)W, \
-                                  (TO*)out, ldo, offsets, sorted, E, N, K, a_div, out_by_pair, gated, limit, alpha, uact)); \
+                                  (TO*)out, ldo, offsets, sorted, E, N, K, a_div, out_by_pair, gated, limit, alpha, uact, SELF)); \
         } while (0)
-        if (dtype == MLLM_F32) MLLM_ROWS(float, float, float);
-        else if (dtype == MLLM_BF16 && kind != 1) MLLM_ROWS(__nv_bfloat16, __nv_bfloat16, __nv_bfloat16);
-        else if (dtype == MLLM_BF16) MLLM_ROWS(__nv_bfloat16, __nv_bfloat16, float);
+        if (dtype == MLLM_F32) MLLM_ROWS(float, float, float, sf);
+        else if (dtype == MLLM_BF16 && kind != 1) MLLM_ROWS(__nv_bfloat16, __nv_bfloat16, __nv_bfloat16, sb);
+        else if (dtype == MLLM_BF16) MLLM_ROWS(__nv_bfloat16, __nv_bfloat16, float, sb);
         else return mllm_fail(1, "moe_grouped: unknown dtype code %d", dtype);
 #undef MLLM_ROWS
         return 0;
     }
     if (dtype == MLLM_BF16 && K % 8 == 0 && lda % 8 == 0 && (uintptr_t)A % 16 == 0 && (uintptr_t)W % 16 == 0) {
-        const dim3 mg((n_pairs + GM - 1) / GM + E, (N + GN - 1) / GN);
+        const dim3 mg((n_pairs + GM - 1) / GM + E + id_tile, (N + GN - 1) / GN);
         if (kind == 0) {
             constexpr size_t smem = (size_t)2 * (GM + 2 * GN) * GROW * 2;
             static bool raised = false;
@@ -612,29 +724,29 @@ MLLM_EXPORT int mllm_moe_grouped(const void* A, long long lda, const void* W, vo
             }
             MLLM_CUDA(mllm_launch(moe_grouped_mma_kernel<__nv_bfloat16, 1>, mg, dim3(128), smem, stream, true, (const __nv_bfloat16*)A,
                                   lda, (const __nv_bfloat16*)W, (__nv_bfloat16*)out, ldo, offsets, sorted, E, N, K, a_div, out_by_pair, act, limit,
-                                  alpha));
+                                  alpha, sb));
         } else if (kind == 2) {
             constexpr size_t smem = (size_t)2 * (GM + GN) * GROW * 2;
             MLLM_CUDA(mllm_launch(moe_grouped_mma_kernel<__nv_bfloat16, 0>, mg, dim3(128), smem, stream, true, (const __nv_bfloat16*)A, lda,
-                                  (const __nv_bfloat16*)W, (__nv_bfloat16*)out, ldo, offsets, sorted, E, N, K, a_div, out_by_pair, act, 0.f, 0.f));
+                                  (const __nv_bfloat16*)W, (__nv_bfloat16*)out, ldo, offsets, sorted, E, N, K, a_div, out_by_pair, act, 0.f, 0.f, sb));
         } else {
             constexpr size_t smem = (size_t)2 * (GM + GN) * GROW * 2;
             MLLM_CUDA(mllm_launch(moe_grouped_mma_kernel<float, 0>, mg, dim3(128), smem, stream, true, (const __nv_bfloat16*)A, lda,
-                                  (const __nv_bfloat16*)W, (float*)out, ldo, offsets, sorted, E, N, K, a_div, out_by_pair, 0, 0.f, 0.f));
+                                  (const __nv_bfloat16*)W, (float*)out, ldo, offsets, sorted, E, N, K, a_div, out_by_pair, 0, 0.f, 0.f, sb));
         }
         return 0;
     }
     if (dtype == MLLM_F32)
         MLLM_CUDA(mllm_launch(moe_grouped_kernel<float, float, float>, grid, block, 0, stream, true, (const float*)A, lda,
-                              (const float*)W, (float*)out, ldo, offsets, sorted, E, N, K, a_div, out_by_pair, gated, limit, alpha, uact));
+                              (const float*)W, (float*)out, ldo, offsets, sorted, E, N, K, a_div, out_by_pair, gated, limit, alpha, uact, sf));
     else if (dtype == MLLM_BF16 && kind != 1)
         MLLM_CUDA(mllm_launch(moe_grouped_kernel<__nv_bfloat16, __nv_bfloat16, __nv_bfloat16>, grid, block, 0, stream, true,
                               (const __nv_bfloat16*)A, lda, (const __nv_bfloat16*)W, (__nv_bfloat16*)out, ldo, offsets, sorted, E,
-                              N, K, a_div, out_by_pair, gated, limit, alpha, uact));
+                              N, K, a_div, out_by_pair, gated, limit, alpha, uact, sb));
     else if (dtype == MLLM_BF16)
         MLLM_CUDA(mllm_launch(moe_grouped_kernel<__nv_bfloat16, __nv_bfloat16, float>, grid, block, 0, stream, true,
                               (const __nv_bfloat16*)A, lda, (const __nv_bfloat16*)W, (float*)out, ldo, offsets, sorted, E, N, K,
-                              a_div, out_by_pair, gated, limit, alpha, uact));
+                              a_div, out_by_pair, gated, limit, alpha, uact, sb));
     else
         return mllm_fail(1, "moe_grouped: unknown dtype code %d", dtype);
     return 0;

@@ -103,25 +103,27 @@ int launch(const float* x, long long x_stride, const int* rows, const float* w1,
     return 0;
 }
 
-// out[t][c] = act(gu[t][c]) * gu[t][F + c]: the gate and the up half of one product's output.
+// out[t][c] = act(gu[t][c]) * gu[t][F + c] (* row_scale[t]): the gate and the up half of one product's output.
 template <typename T>
 __global__ void __launch_bounds__(256)
 gated_act_kernel(const T* gu, long long gu_stride, T* __restrict__ out, long long out_stride, int rows, int F, int act,
-                 float limit, float alpha) {
+                 float limit, float alpha, const float* row_scale) {
     pdl_wait();
     pdl_launch();
     const long long total = (long long)rows * F;
     for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
         const int t = (int)(i / F), c = (int)(i % F);
         const float g = to_f32(gu[(size_t)t * gu_stride + c]), u = to_f32(gu[(size_t)t * gu_stride + F + c]);
-        out[(size_t)t * out_stride + c] = from_f32<T>(gate_mul(g, u, act, limit, alpha));
+        const float v = gate_mul(g, u, act, limit, alpha);
+        out[(size_t)t * out_stride + c] = from_f32<T>(row_scale ? v * row_scale[t] : v);
     }
 }
 
 // x[r] += (v / sqrt(mean(v^2) + eps) * w) * ls with v = y[r] (+ sum_k pw[r][k] * pairs[r * top + k], the weighted
 // results of a routed feed-forward's chosen experts, in the order of k): a branch's result, normed, scaled per column and
 // added to the 32-bit residual stream in one pass (ls, y or the pairs may be absent).  With `nw` the new x is normed once
-// more, h = x / sqrt(mean(x^2) + neps) * (nw + noff), for the branch that reads it next.  The row is kept in shared memory.
+// more, h = x / sqrt(mean(x^2) + neps) * (nw + noff), for the branch that reads it next; with h alone it is copied there as
+// it is.  The row is kept in shared memory.
 template <typename TOut>
 __global__ void __launch_bounds__(256)
 join_kernel(const float* y, long long y_stride, const float* pairs, const float* pw, int top, const float* __restrict__ w,
@@ -151,9 +153,13 @@ join_kernel(const float* y, long long y_stride, const float* pairs, const float*
         rowbuf[d] = v;
         q2 = fmaf(v, v, q2);
     }
-    if (!nw) return;
-    const float r2 = sqrtf(block_sum(q2, scratch) / (float)D + neps);
+    if (!h) return;
     TOut* hr = h + r * h_stride;
+    if (!nw) {                              // a plain copy: each thread reads what it wrote itself
+        for (int d = threadIdx.x; d < D; d += blockDim.x) hr[d] = from_f32<TOut>(rowbuf[d]);
+        return;
+    }
+    const float r2 = sqrtf(block_sum(q2, scratch) / (float)D + neps);
     for (int d = threadIdx.x; d < D; d += blockDim.x) hr[d] = from_f32<TOut>(rowbuf[d] / r2 * (nw[d] + noff));
 }
 
@@ -230,7 +236,8 @@ MLLM_EXPORT int mllm_norm_scale_add(const float* y, long long y_stride, const fl
         MLLM_CUDA(cudaFuncSetAttribute(join_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
         raised = true;
     }
-    if (nw && h_dtype == MLLM_BF16)
+    if (nw && !h) return mllm_fail(1, "norm_scale_add: a second norm without a place for its result");
+    if (h && h_dtype == MLLM_BF16)
         MLLM_CUDA(mllm_launch(join_kernel<__nv_bfloat16>, dim3(R), dim3(threads), smem, stream, true, y, y_stride, pairs, pw, top,
                               w, ls, x, x_stride, nw, noff, neps, (__nv_bfloat16*)h, h_stride, D, eps));
     else
@@ -254,16 +261,16 @@ MLLM_EXPORT int mllm_rmsnorm(const float* x, long long x_stride, const int* rows
 }
 
 MLLM_EXPORT int mllm_gated_act(const void* gu, long long gu_stride, void* out, long long out_stride, int rows, int F,
-                               int act, float limit, float alpha, int dtype, cudaStream_t stream) {
+                               int act, float limit, float alpha, const float* row_scale, int dtype, cudaStream_t stream) {
     if (rows <= 0 || F <= 0) return 0;
     const long long total = (long long)rows * F;
     const int grid = (int)((total + 255) / 256 < 8192 ? (total + 255) / 256 : 8192);
     if (dtype == MLLM_F32)
         MLLM_CUDA(mllm_launch(gated_act_kernel<float>, dim3(grid), dim3(256), 0, stream, true, (const float*)gu, gu_stride,
-                              (float*)out, out_stride, rows, F, act, limit, alpha));
+                              (float*)out, out_stride, rows, F, act, limit, alpha, row_scale));
     else if (dtype == MLLM_BF16)
         MLLM_CUDA(mllm_launch(gated_act_kernel<__nv_bfloat16>, dim3(grid), dim3(256), 0, stream, true,
-                              (const __nv_bfloat16*)gu, gu_stride, (__nv_bfloat16*)out, out_stride, rows, F, act, limit, alpha));
+                              (const __nv_bfloat16*)gu, gu_stride, (__nv_bfloat16*)out, out_stride, rows, F, act, limit, alpha, row_scale));
     else
         return mllm_fail(1, "gated_act: unknown dtype code %d", dtype);
     return 0;

@@ -1,0 +1,306 @@
+// The selective scan with a state per channel (Mamba's first form).  Per channel c and state entry n, S zero at the start:
+//   dt_c = softplus(raw_c + bias_c)
+//   S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n          A negative: [C, N] rates
+//   y_c = sum_n S[c, n] C_n + skip_c x_c                          out_c = out_scale * y_c * silu(z_c)
+// x (the convolution's output), B, C and z come in the activation dtype; dt, the decays, the state and the sums are 32-bit.
+//
+// `scan` (prompt portions): a CTA of 128 threads takes 128 / L channels of one request; L lanes share a channel and keep R
+// consecutive state entries each in registers for the whole walk.  Tokens come 16 (8) at a time: the next chunk's inputs
+// are fetched into registers while this one is walked, softplus is taken once per (token, channel) on the way to shared
+// memory, the gate on the way out.  The decays do not depend on the state, so only one fused multiply-add per entry is
+// sequential.  `step` (single tokens): the step size's projection, softplus, update, output and gate in one launch; S, A and
+// the projection's weights are read before the kernel waits for its predecessor.
+// Every state entry is a recurrence of its own and both kernels do the same operations per token, so the state after some
+// tokens is the same bits however they were cut into portions (single tokens make dt in another summation order).
+#include "common.cuh"
+
+namespace {
+
+constexpr int THREADS = 128;
+constexpr float LOG2E = 1.4426950408889634f;
+
+struct SelArgs {
+    const float* A;                 // [C][N]
+    const float* skip;              // [C]
+    const float* bias;              // [C] of the step sizes
+    float* state;                   // [slots][stride]: S [C][N] at the row's start
+    long long stride;
+    const int* cu_q;
+    const int* slots;
+    int C, N, write_state;
+    float out_scale;
+};
+
+__device__ __forceinline__ float softplus_f(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
+__device__ __forceinline__ float silu_f(float v) { return v / (1.0f + expf(-v)); }
+
+// exp(dt * a): on the bfloat16 path the rates are kept in units of ln 2 and the exponential is one instruction
+template <typename T> __device__ __forceinline__ float rate_unit() { return sizeof(T) == 4 ? 1.0f : LOG2E; }
+template <typename T> __device__ __forceinline__ float decay_of(float dt, float a) {
+    if constexpr (sizeof(T) == 4) return expf(dt * a);
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(dt * a));
+    return y;
+}
+
+template <typename T, int R>
+__device__ __forceinline__ float advance(float* s, const float* ar, float dt, float dx, const float* b, const float* c) {
+    float acc = 0.f;
+#pragma unroll
+    for (int i = 0; i < R; i += 4) {
+        const float4 bv = *reinterpret_cast<const float4*>(b + i), cv = *reinterpret_cast<const float4*>(c + i);
+        s[i] = fmaf(decay_of<T>(dt, ar[i]), s[i], dx * bv.x);
+        s[i + 1] = fmaf(decay_of<T>(dt, ar[i + 1]), s[i + 1], dx * bv.y);
+        s[i + 2] = fmaf(decay_of<T>(dt, ar[i + 2]), s[i + 2], dx * bv.z);
+        s[i + 3] = fmaf(decay_of<T>(dt, ar[i + 3]), s[i + 3], dx * bv.w);
+        acc += (s[i] * cv.x + s[i + 1] * cv.y) + (s[i + 2] * cv.z + s[i + 3] * cv.w);
+    }
+    return acc;
+}
+
+template <int L>
+__device__ __forceinline__ float lanes_sum(float v) {
+#pragma unroll
+    for (int o = L / 2; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    return v;
+}
+
+// grid (channel blocks, requests).  x [T][ldx], raw step sizes dt [T][lddt] (32-bit, bias not yet added), bc [T][ldbc] with
+// B at b_off and C at c_off, z [T][ldz], out [T][ldo].
+template <typename T, int L, int R>
+__global__ void __launch_bounds__(THREADS)
+selective_scan_kernel(const T* x, long long ldx, const float* dt, long long lddt, const T* bc, long long ldbc, int b_off,
+                      int c_off, const T* z, long long ldz, T* __restrict__ out, long long ldo, SelArgs a) {
+    constexpr int CPB = THREADS / L, NR = L * R, CH = NR > 128 ? 8 : 16;
+    constexpr int NB = (CH * NR + THREADS - 1) / THREADS, NX = (CH * CPB + THREADS - 1) / THREADS;
+    __shared__ __align__(16) float Bs[2][CH * NR], Cs[2][CH * NR];
+    __shared__ float xs[2][CH * CPB], ds[2][CH * CPB], ys[CH * CPB];
+    const int tid = threadIdx.x, seq = blockIdx.y, base = blockIdx.x * CPB;
+    const int ch = tid / L, lane = tid % L, c = base + ch;
+    const bool live = c < a.C;
+    float ar[R], s[R];
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+        const int r = lane * R + i;
+        ar[i] = live && r < a.N ? a.A[(size_t)c * a.N + r] * rate_unit<T>() : 0.f;
+    }
+    const float skip = live ? a.skip[c] : 0.f;
+    pdl_wait();
+    pdl_launch();
+    const int t0 = a.cu_q[seq], n = a.cu_q[seq + 1] - t0;
+    if (n <= 0) return;
+    float* S = a.state + (size_t)a.slots[seq] * a.stride + (size_t)c * a.N;
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+        const int r = lane * R + i;
+        s[i] = live && r < a.N ? S[r] : 0.f;
+    }
+    T rb[NB], rc[NB], rx[NX], rz[NX], rz_next[NX];
+    float rd[NX];
+    auto fetch = [&](int c0) {
+        const int nc = min(CH, n - c0);
+#pragma unroll
+        for (int u = 0; u < NB; ++u) {
+            const int i = tid + u * THREADS, tt = i / NR, r = i % NR;
+            const bool ok = i < CH * NR && tt < nc && r < a.N;
+            const T* row = bc + (size_t)(t0 + c0 + (ok ? tt : 0)) * ldbc;
+            rb[u] = ok ? row[b_off + r] : from_f32<T>(0.f);
+            rc[u] = ok ? row[c_off + r] : from_f32<T>(0.f);
+        }
+#pragma unroll
+        for (int u = 0; u < NX; ++u) {
+            const int i = tid + u * THREADS, tt = i / CPB, cc = base + i % CPB;
+            const bool ok = i < CH * CPB && tt < nc && cc < a.C;
+            const size_t t = t0 + c0 + (ok ? tt : 0);
+            rx[u] = ok ? x[t * ldx + cc] : from_f32<T>(0.f);
+            rz_next[u] = ok ? z[t * ldz + cc] : from_f32<T>(0.f);
+            rd[u] = ok ? dt[t * lddt + cc] + a.bias[cc] : 0.f;
+        }
+    };
+    auto put = [&](int buf) {
+#pragma unroll
+        for (int u = 0; u < NB; ++u) {
+            const int i = tid + u * THREADS;
+            if (i < CH * NR) { Bs[buf][i] = to_f32(rb[u]); Cs[buf][i] = to_f32(rc[u]); }
+        }
+#pragma unroll
+        for (int u = 0; u < NX; ++u) {
+            const int i = tid + u * THREADS;
+            if (i < CH * CPB) { xs[buf][i] = to_f32(rx[u]); ds[buf][i] = softplus_f(rd[u]); }
+        }
+    };
+    fetch(0);
+    put(0);
+    for (int c0 = 0, buf = 0; c0 < n; c0 += CH, buf ^= 1) {
+        const int nc = min(CH, n - c0);
+#pragma unroll
+        for (int u = 0; u < NX; ++u) rz[u] = rz_next[u];
+        __syncthreads();                        // this chunk is in; the other buffer and ys are free
+        const bool more = c0 + CH < n;
+        if (more) fetch(c0 + CH);
+        auto walk = [&](int tt) {
+            const float d = ds[buf][tt * CPB + ch], xv = xs[buf][tt * CPB + ch];
+            const float acc = lanes_sum<L>(advance<T, R>(s, ar, d, d * xv, &Bs[buf][tt * NR + lane * R], &Cs[buf][tt * NR + lane * R]));
+            if (lane == 0) ys[tt * CPB + ch] = fmaf(skip, xv, acc);
+        };
+        if (nc == CH) {
+#pragma unroll 4
+            for (int tt = 0; tt < CH; ++tt) walk(tt);
+        } else {
+            for (int tt = 0; tt < nc; ++tt) walk(tt);
+        }
+        if (more) put(buf ^ 1);
+        __syncthreads();
+#pragma unroll
+        for (int u = 0; u < NX; ++u) {
+            const int i = tid + u * THREADS, tt = i / CPB, cc = base + i % CPB;
+            if (i < CH * CPB && tt < nc && cc < a.C)
+                out[(size_t)(t0 + c0 + tt) * ldo + cc] = from_f32<T>(ys[i] * silu_f(to_f32(rz[u])) * a.out_scale);
+        }
+    }
+    if (a.write_state && live) {
+#pragma unroll
+        for (int i = 0; i < R; ++i)
+            if (lane * R + i < a.N) S[lane * R + i] = s[i];
+    }
+}
+
+// Single tokens: grid (channel blocks, requests).  low [T][ldlow]: the step sizes' low-rank columns (rank), B at b_off, C at
+// c_off; W [C][rank8], rank8 the rank rounded up to 8, zeros beyond the rank.
+template <typename T, int L, int R>
+__global__ void __launch_bounds__(THREADS)
+selective_step_kernel(const T* x, long long ldx, const T* low, long long ldlow, int rank, int b_off, int c_off,
+                      const T* __restrict__ W, const T* z, long long ldz, T* __restrict__ out, long long ldo, SelArgs a) {
+    constexpr int CPB = THREADS / L, NR = L * R, V = 16 / sizeof(T);
+    extern __shared__ __align__(16) float lows[];               // [rank8]
+    __shared__ __align__(16) float Bs[NR], Cs[NR];
+    const int tid = threadIdx.x, seq = blockIdx.y;
+    const int ch = tid / L, lane = tid % L, c = blockIdx.x * CPB + ch;
+    const int rank8 = (rank + 7) / 8 * 8;
+    const bool live = c < a.C;
+    const int t = a.cu_q[seq];
+    float* S = a.state + (size_t)a.slots[seq] * a.stride + (size_t)c * a.N;
+    float ar[R], s[R];
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+        const int r = lane * R + i;
+        const bool ok = live && r < a.N;
+        ar[i] = ok ? a.A[(size_t)c * a.N + r] * rate_unit<T>() : 0.f;
+        s[i] = ok ? S[r] : 0.f;
+    }
+    const T* wr = W + (size_t)(live ? c : 0) * rank8;
+    uint4 first = make_uint4(0u, 0u, 0u, 0u);
+    if (lane * V < rank8) first = *reinterpret_cast<const uint4*>(wr + lane * V);
+    const float skip = live ? a.skip[c] : 0.f, bias = live ? a.bias[c] : 0.f;
+    pdl_wait();
+    pdl_launch();
+    const T* lr = low + (size_t)t * ldlow;
+    for (int r = tid; r < rank8; r += THREADS) lows[r] = r < rank ? to_f32(lr[r]) : 0.f;
+    for (int r = tid; r < NR; r += THREADS) {
+        Bs[r] = r < a.N ? to_f32(lr[b_off + r]) : 0.f;
+        Cs[r] = r < a.N ? to_f32(lr[c_off + r]) : 0.f;
+    }
+    const float xv = live ? to_f32(x[(size_t)t * ldx + c]) : 0.f;
+    const float zv = live && lane == 0 ? to_f32(z[(size_t)t * ldz + c]) : 0.f;
+    __syncthreads();
+    float acc = 0.f;
+    for (int r = lane * V; r < rank8; r += L * V) {
+        const uint4 w4 = r == lane * V ? first : *reinterpret_cast<const uint4*>(wr + r);
+        const T* w = reinterpret_cast<const T*>(&w4);
+#pragma unroll
+        for (int e = 0; e < V; ++e) acc = fmaf(to_f32(w[e]), lows[r + e], acc);
+    }
+    const float d = softplus_f(lanes_sum<L>(acc) + bias);
+    const float y = lanes_sum<L>(advance<T, R>(s, ar, d, d * xv, Bs + lane * R, Cs + lane * R));
+    if (!live) return;
+    if (lane == 0) out[(size_t)t * ldo + c] = from_f32<T>(fmaf(skip, xv, y) * silu_f(zv) * a.out_scale);
+    if (a.write_state) {
+#pragma unroll
+        for (int i = 0; i < R; ++i)
+            if (lane * R + i < a.N) S[lane * R + i] = s[i];
+    }
+}
+
+int check(const char* what, const SelArgs& a, int S) {
+    if (a.C <= 0 || a.N <= 0 || a.N > 256) return mllm_fail(1, "%s: %d channels with states of %d entries (at most 256)", what, a.C, a.N);
+    if (a.stride < (long long)a.C * a.N) return mllm_fail(1, "%s: state rows of %lld floats", what, a.stride);
+    if (S > 65535) return mllm_fail(1, "%s: more than 65535 requests in a step", what);
+    return 0;
+}
+
+// lanes per channel, so that L * 4 (or 32 * 8) entries cover the state
+int lanes_for(int N) {
+    int L = 1;
+    while (L < 32 && L * 4 < N) L *= 2;
+    return L;
+}
+
+#define MLLM_BY_LANES(GO)                                                                                                \
+    do {                                                                                                                 \
+        switch (lanes_for(a.N)) {                                                                                        \
+            case 1: GO(1, 4); break;                                                                                     \
+            case 2: GO(2, 4); break;                                                                                     \
+            case 4: GO(4, 4); break;                                                                                     \
+            case 8: GO(8, 4); break;                                                                                     \
+            case 16: GO(16, 4); break;                                                                                   \
+            default: if (a.N <= 128) GO(32, 4); else GO(32, 8);                                                          \
+        }                                                                                                                \
+    } while (0)
+
+template <typename T>
+int scan_launch(const void* x, long long ldx, const float* dt, long long lddt, const void* bc, long long ldbc, int b_off, int c_off,
+                const void* z, long long ldz, void* out, long long ldo, int S, const SelArgs& a, cudaStream_t stream) {
+#define MLLM_GO(L, R)                                                                                                    \
+    MLLM_CUDA(mllm_launch(selective_scan_kernel<T, L, R>, dim3((a.C + THREADS / L - 1) / (THREADS / L), S), dim3(THREADS), 0, \
+                          stream, true, (const T*)x, ldx, dt, lddt, (const T*)bc, ldbc, b_off, c_off, (const T*)z, ldz,  \
+                          (T*)out, ldo, a))
+    MLLM_BY_LANES(MLLM_GO);
+#undef MLLM_GO
+    return 0;
+}
+
+template <typename T>
+int step_launch(const void* x, long long ldx, const void* low, long long ldlow, int rank, int b_off, int c_off, const void* W,
+                const void* z, long long ldz, void* out, long long ldo, int S, const SelArgs& a, cudaStream_t stream) {
+    const size_t smem = (size_t)((rank + 7) / 8 * 8) * 4;
+#define MLLM_GO(L, R)                                                                                                    \
+    MLLM_CUDA(mllm_launch(selective_step_kernel<T, L, R>, dim3((a.C + THREADS / L - 1) / (THREADS / L), S), dim3(THREADS), smem, \
+                          stream, true, (const T*)x, ldx, (const T*)low, ldlow, rank, b_off, c_off, (const T*)W, (const T*)z, \
+                          ldz, (T*)out, ldo, a))
+    MLLM_BY_LANES(MLLM_GO);
+#undef MLLM_GO
+    return 0;
+}
+
+}  // namespace
+
+MLLM_EXPORT int mllm_selective_max_state() { return 256; }
+MLLM_EXPORT int mllm_selective_max_rank() { return 10240; }
+
+MLLM_EXPORT int mllm_selective_scan(const void* x, long long ldx, const float* dt, long long lddt, const void* bc, long long ldbc,
+                                    int b_off, int c_off, const void* z, long long ldz, const float* A, const float* skip,
+                                    const float* bias, float* state, long long stride, const int* cu_q, const int* slots, void* out,
+                                    long long ldo, int S, int C, int N, float out_scale, int write_state, int dtype,
+                                    cudaStream_t stream) {
+    if (S <= 0) return 0;
+    SelArgs a{A, skip, bias, state, stride, cu_q, slots, C, N, write_state, out_scale};
+    if (int rc = check("selective_scan", a, S)) return rc;
+    if (dtype == MLLM_F32) return scan_launch<float>(x, ldx, dt, lddt, bc, ldbc, b_off, c_off, z, ldz, out, ldo, S, a, stream);
+    if (dtype == MLLM_BF16) return scan_launch<__nv_bfloat16>(x, ldx, dt, lddt, bc, ldbc, b_off, c_off, z, ldz, out, ldo, S, a, stream);
+    return mllm_fail(1, "selective_scan: unknown dtype code %d", dtype);
+}
+
+MLLM_EXPORT int mllm_selective_step(const void* x, long long ldx, const void* low, long long ldlow, int rank, int b_off, int c_off,
+                                    const void* W, const void* z, long long ldz, const float* A, const float* skip,
+                                    const float* bias, float* state, long long stride, const int* cu_q, const int* slots, void* out,
+                                    long long ldo, int S, int C, int N, float out_scale, int write_state, int dtype,
+                                    cudaStream_t stream) {
+    if (S <= 0) return 0;
+    SelArgs a{A, skip, bias, state, stride, cu_q, slots, C, N, write_state, out_scale};
+    if (int rc = check("selective_step", a, S)) return rc;
+    if (rank <= 0 || rank > mllm_selective_max_rank()) return mllm_fail(1, "selective_step: step sizes of rank %d", rank);
+    if ((uintptr_t)W % 16) return mllm_fail(1, "selective_step: the projection's rows must start on 16 bytes");
+    if (dtype == MLLM_F32) return step_launch<float>(x, ldx, low, ldlow, rank, b_off, c_off, W, z, ldz, out, ldo, S, a, stream);
+    if (dtype == MLLM_BF16) return step_launch<__nv_bfloat16>(x, ldx, low, ldlow, rank, b_off, c_off, W, z, ldz, out, ldo, S, a, stream);
+    return mllm_fail(1, "selective_step: unknown dtype code %d", dtype);
+}

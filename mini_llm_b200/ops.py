@@ -41,7 +41,8 @@ def _signatures(lib):
     lib.mllm_set_pdl.argtypes = [c_int]
     lib.mllm_set_pdl.restype = c_int
     sig = {
-        "mllm_embed": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p],
+        "mllm_token_side_gate": [c_void_p, c_ll, c_void_p, c_void_p, c_ll, c_int, c_void_p, c_ll, c_int, c_int, c_int, c_void_p],
+        "mllm_embed": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p],
         "mllm_concat_terms": [c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_ll, c_int, c_int, c_int, c_int, c_void_p],
         "mllm_resolve_tokens": [c_void_p, c_int, c_void_p, c_int, c_void_p],
         "mllm_layernorm": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_void_p],
@@ -92,7 +93,7 @@ def _signatures(lib):
         "mllm_gated_recurrence_wide": [c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_void_p, c_void_p,
                                        c_void_p, c_void_p, c_void_p, c_ll, c_int, c_int, c_int, c_int, c_int, c_int,
                                        c_void_p],
-        "mllm_gated_act": [c_void_p, c_ll, c_void_p, c_ll, c_int, c_int, c_int, c_float, c_float, c_int, c_void_p],
+        "mllm_gated_act": [c_void_p, c_ll, c_void_p, c_ll, c_int, c_int, c_int, c_float, c_float, c_void_p, c_int, c_void_p],
         "mllm_paged_write": [c_void_p, c_ll, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
         "mllm_paged_write_kv": [c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
                                 c_int, c_int, c_void_p],
@@ -100,7 +101,7 @@ def _signatures(lib):
         "mllm_attention_bias": [c_void_p, c_ll, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
                                 c_void_p, c_ll, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                                 c_float, c_float, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_float, c_void_p, c_int,
-                                c_int, c_void_p],
+                                c_void_p, c_ll, c_int, c_int, c_void_p],
         "mllm_qk_norm_rope": [c_void_p, c_ll, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float,
                               c_void_p, c_int, c_int, c_void_p, c_void_p, c_ll, c_void_p, c_void_p, c_int, c_void_p, c_int,
                               c_int, c_void_p, c_ll, c_void_p, c_void_p, c_ll, c_int, c_int, c_void_p],
@@ -138,7 +139,7 @@ def _signatures(lib):
                                       c_int, c_int, c_int, c_float, c_void_p, c_void_p],
         "mllm_latent_mma_ok": [c_int, c_int, c_int],
         "mllm_ssd_conv": [c_void_p, c_ll, c_int, c_void_p, c_void_p, c_void_p, c_ll, c_int, c_void_p, c_void_p, c_void_p,
-                          c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+                          c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
         "mllm_ssd_scan": [c_void_p, c_int, c_int, c_int, c_void_p, c_ll, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_ll,
                           c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
         "mllm_gated_group_norm": [c_void_p, c_void_p, c_ll, c_void_p, c_void_p, c_ll, c_int, c_int, c_int, c_float, c_int,
@@ -158,9 +159,21 @@ def _signatures(lib):
         "mllm_mlstm_step": [c_void_p, c_ll, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_ll, c_void_p, c_void_p, c_void_p,
                             c_void_p, c_ll, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_float, c_int, c_int, c_void_p],
         "mllm_moe_route": [c_void_p, c_ll, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
-                           c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
+                           c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
         "mllm_moe_grouped": [c_void_p, c_ll, c_void_p, c_void_p, c_ll, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                             c_int, c_int, c_int, c_float, c_float, c_int, c_void_p],
+                             c_int, c_int, c_int, c_float, c_float, c_void_p, c_ll, c_int, c_int, c_int, c_void_p],
+        "mllm_retention_step_ok": [c_int, c_int],
+        "mllm_rotate_heads": [c_void_p, c_ll, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_float, c_void_p, c_int, c_void_p],
+        "mllm_retention_scan": [c_void_p, c_ll, c_int, c_int, c_int, c_void_p, c_void_p, c_ll, c_void_p, c_void_p, c_void_p, c_int,
+                                c_int, c_int, c_int, c_int, c_int, c_void_p],
+        "mllm_retention_finish": [c_void_p, c_void_p, c_ll, c_int, c_void_p, c_ll, c_int, c_int, c_int, c_float, c_int, c_void_p],
+        "mllm_retention_step": [c_void_p, c_ll, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p,
+                                c_ll, c_void_p, c_void_p, c_void_p, c_ll, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p],
+        "mllm_selective_scan": [c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_ll, c_int, c_int, c_void_p, c_ll, c_void_p, c_void_p, c_void_p,
+                                c_void_p, c_ll, c_void_p, c_void_p, c_void_p, c_ll, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p],
+        "mllm_selective_step": [c_void_p, c_ll, c_void_p, c_ll, c_int, c_int, c_int, c_void_p, c_void_p, c_ll, c_void_p, c_void_p,
+                                c_void_p, c_void_p, c_ll, c_void_p, c_void_p, c_void_p, c_ll, c_int, c_int, c_int, c_float, c_int, c_int,
+                                c_void_p],
         "mllm_moe_combine": [c_void_p, c_void_p, c_void_p, c_ll, c_int, c_int, c_int, c_int, c_void_p],
         "mllm_argmax": [c_void_p, c_ll, c_int, c_int, c_void_p, c_void_p],
         "mllm_argmax_sliced": [c_void_p, c_ll, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
@@ -354,10 +367,11 @@ def _rows(name: str, t: torch.Tensor):
 
 
 # --------------------------------------------------------------------------- embedding
-def embed(ids, positions, table, pos_table, out, copies: int = 1, scale: float = 1.0, keep=None) -> None:
+def embed(ids, positions, table, pos_table, out, copies: int = 1, scale: float = 1.0, keep=None, act=None) -> None:
     """out[t] = table[ids[t]] * scale (+ pos_table[positions[t]]), 32-bit; with ``copies`` > 1 a row of out holds that many
     copies of the token's row side by side (a residual of several streams at its start).  ``keep`` (32-bit [T, D]): the
-    row once more, for a part that reads it later in the step."""
+    row once more, for a part that reads it later in the step.  ``act`` [T, D]: likewise in the table's dtype, for the
+    products of a layer that reads the residual itself."""
     _cuda("ids", ids, torch.int32)
     _cuda("table", table)
     _cuda("out", out, torch.float32)
@@ -371,6 +385,10 @@ def embed(ids, positions, table, pos_table, out, copies: int = 1, scale: float =
         _cuda("keep", keep, torch.float32)
         if tuple(keep.shape) != (T, D):
             raise KernelError(f"embed: keep {tuple(keep.shape)} for {T} rows of {D}")
+    if act is not None:
+        _cuda("act", act, table.dtype)
+        if tuple(act.shape) != (T, D):
+            raise KernelError(f"embed: act {tuple(act.shape)} for {T} rows of {D}")
     pp = None
     if pos_table is not None:
         _cuda("positions", positions, torch.int32)
@@ -379,8 +397,22 @@ def embed(ids, positions, table, pos_table, out, copies: int = 1, scale: float =
             raise KernelError("embed: position table or positions do not fit")
         pp = pos_table.data_ptr()
     _call("mllm_embed", ids.data_ptr(), positions.data_ptr() if pos_table is not None else None,
-          table.data_ptr(), pp, out.data_ptr(), keep.data_ptr() if keep is not None else None, T, D, int(copies), float(scale),
+          table.data_ptr(), pp, out.data_ptr(), keep.data_ptr() if keep is not None else None,
+          act.data_ptr() if act is not None else None, T, D, int(copies), float(scale),
           _dt(table), _stream())
+
+
+def token_side_gate(z, ids, table, off: int, out) -> None:
+    """out[t, c] = gelu_tanh(z[t, c]) * table[ids[t], off + c]: z 32-bit [T, d], table [vocab, .] and out [T, d] in one dtype."""
+    _cuda("z", z, torch.float32, contiguous=False)
+    _cuda("ids", ids, torch.int32)
+    _cuda("table", table)
+    _cuda("out", out, table.dtype, contiguous=False)
+    T, d = z.shape
+    if ids.numel() != T or tuple(out.shape) != (T, d) or off < 0 or off + d > table.shape[1]:
+        raise KernelError(f"token_side_gate: z {tuple(z.shape)}, table {tuple(table.shape)} from column {off}, out {tuple(out.shape)}")
+    _call("mllm_token_side_gate", z.data_ptr(), _rows("z", z), ids.data_ptr(), table.data_ptr(), table.shape[1], int(off),
+          out.data_ptr(), _rows("out", out), T, d, _dt(table), _stream())
 
 
 def concat_terms(x, x0, out, terms: int) -> None:
@@ -460,10 +492,10 @@ def rmsnorm(x, weight, eps: float, out, rows=None, unit_offset: bool = True, wei
           float(scale), _dt(out), _stream())
 
 
-def gated_act(gu, out, act: str, limit: float = 0.0, alpha: float = 1.0) -> None:
+def gated_act(gu, out, act: str, limit: float = 0.0, alpha: float = 1.0, row_scale=None) -> None:
     """out[t, c] = act(gu[t, c]) * gu[t, F + c] for gu [T, 2F]: the gate and the up half of one product.
     ``act`` "swiglu_clamp": with g the gate cut off above ``limit`` and u the up value cut off at +-``limit``,
-    out = g * sigmoid(alpha * g) * (u + 1)."""
+    out = g * sigmoid(alpha * g) * (u + 1).  ``row_scale`` (float32 [T]): a factor per row on the result."""
     _cuda("gu", gu, contiguous=False)
     _cuda("out", out, gu.dtype, contiguous=False)
     T, F = out.shape
@@ -473,8 +505,12 @@ def gated_act(gu, out, act: str, limit: float = 0.0, alpha: float = 1.0) -> None
         raise KernelError(f"gated_act: unknown activation {act!r}; known: {sorted(_GATE_ACT)}")
     if act == "swiglu_clamp" and not limit > 0:
         raise KernelError("gated_act: the clamped form needs a positive limit")
+    if row_scale is not None:
+        _cuda("row_scale", row_scale, torch.float32)
+        if row_scale.numel() != T:
+            raise KernelError("gated_act: one factor per row")
     _call("mllm_gated_act", gu.data_ptr(), _rows("gu", gu), out.data_ptr(), _rows("out", out), T, F, _GATE_ACT[act],
-          float(limit), float(alpha), _dt(gu), _stream())
+          float(limit), float(alpha), row_scale.data_ptr() if row_scale is not None else None, _dt(gu), _stream())
 
 
 # --------------------------------------------------------------------------- linear
@@ -847,7 +883,7 @@ _bias_split_keys = None
 
 def biased_attention(q, k_pages, v_pages, block_table, ctx, out, *, num_heads, num_kv_heads, scale, dist_bias=None,
                      q_scale=None, out_scale: float = 1.0, window=None, chunk=None, sink=None, softcap: float = 0.0,
-                     slopes=None, impl: Optional[str] = None) -> None:
+                     slopes=None, keep_first: int = 0, gate=None, impl: Optional[str] = None) -> None:
     """Causal attention over the cache with keys and values of different sizes, an additive score bias
     ``dist_bias[head, i - j]`` (float32 [heads, n]) and a factor ``q_scale[position]`` (float32 [n]) on the query:
     out[t] = out_scale * softmax_j((q_t . k_j) * scale * q_scale[p_t] + dist_bias[h, p_t - j]) v_j.
@@ -855,6 +891,8 @@ def biased_attention(q, k_pages, v_pages, block_table, ctx, out, *, num_heads, n
     positions [b * chunk, (b + 1) * chunk) of the request); ``sink`` (float32 [heads]): exp(sink[h]) is one more
     term of the softmax's denominator and of nothing else.  ``softcap`` c > 0: the scaled product s becomes
     c * tanh(s / c) before any bias is added; ``slopes`` (float32 [heads]): slopes[h] * (p_t - j) is taken off the score.
+    ``keep_first`` f: the first f positions stay visible beyond the window or the chunk.  ``gate`` [T, heads * dv] in q's
+    dtype: the result is multiplied, entry by entry, with sigmoid(gate).
 
     q [T, heads * dkq], k_pages [P, kv_heads, page_size, dk] with dk >= dkq a multiple of 8 (key rows padded with
     zeros), v_pages [P, kv_heads, page_size, dv], out [T, heads * dv] (rows contiguous; a column slice of a wider
@@ -897,6 +935,10 @@ def biased_attention(q, k_pages, v_pages, block_table, ctx, out, *, num_heads, n
         _cuda("slopes", slopes, torch.float32)
         if slopes.numel() != num_heads:
             raise KernelError("biased_attention: one slope per query head")
+    if gate is not None:
+        _cuda("gate", gate, q.dtype, contiguous=False)
+        if tuple(gate.shape) != (T, num_heads * dv):
+            raise KernelError(f"biased_attention: gate {tuple(gate.shape)} for {num_heads} heads of {dv}")
     if impl is None:
         impl = "simt"
         if getattr(ctx, "decode_only", False):
@@ -930,7 +972,8 @@ def biased_attention(q, k_pages, v_pages, block_table, ctx, out, *, num_heads, n
           float(out_scale), dist_bias.data_ptr() if dist_bias is not None else None, n_dist,
           q_scale.data_ptr() if q_scale is not None else None, int(window or 0), int(chunk or 0),
           sink.data_ptr() if sink is not None else None, float(softcap or 0.0),
-          slopes.data_ptr() if slopes is not None else None, _dt(q), {"simt": 0, "tiled": 1, "split": 2, "mma": 3}[impl],
+          slopes.data_ptr() if slopes is not None else None, int(keep_first), gate.data_ptr() if gate is not None else None,
+          _rows("gate", gate) if gate is not None else 0, _dt(q), {"simt": 0, "tiled": 1, "split": 2, "mma": 3}[impl],
           _stream())
     if impl == "split":
         global launches
@@ -1018,7 +1061,7 @@ def mixed_splits(max_ctx_len: int, window=None) -> int:
 # --------------------------------------------------------------------------- normed and rotated queries and keys
 def qk_norm_rope(proj, q_off: int, k_off: int, v_off: int, ctx, q_out, k_pages, v_pages, slot_mapping, *, heads: int,
                  kv_heads: int, head_dim: int, v_head_dim: int, q_norm=None, k_norm=None, eps: float = 0.0, freq=None,
-                 rot_dims: int = 0, interleaved: bool = True, head_norm: bool = False, v_first=None, v_lambda=None,
+                 rot_dims: int = 0, interleaved: bool = True, head_norm=False, v_first=None, v_lambda=None,
                  v_keep=None) -> None:
     """What stands between a Q | K | V projection and attention when queries and keys are normed and rotated.
 
@@ -1029,7 +1072,8 @@ def qk_norm_rope(proj, q_off: int, k_off: int, v_off: int, ctx, q_out, k_pages, 
     pairs with 2i + 1, else i with i + rot_dims / 2.  Queries go to q_out [T, heads * head_dim]; keys (rows of the
     pages may be padded) and values go to the tokens' slots (``slot_mapping`` None: nothing is cached).  All 32-bit
     up to the final rounding.  ``head_norm`` (instead of q_norm / k_norm): after the rotation every query head and every
-    key head is divided by its own root mean square (eps inside the root, no weights).  ``v_first`` [T, kv_heads *
+    key head is divided by its own root mean square (eps inside the root, no weights); "weighted": before the rotation
+    every query head and every key head is, and multiplied by q_norm or k_norm, which then have head_dim entries.  ``v_first`` [T, kv_heads *
     v_head_dim] with ``v_lambda`` (a float32 scalar on the device): the values become (1 - lambda) v + lambda v_first
     before they are cached; ``v_keep`` [T, kv_heads * v_head_dim] gets the values as they are cached."""
     _cuda("proj", proj, contiguous=False)
@@ -1039,7 +1083,8 @@ def qk_norm_rope(proj, q_off: int, k_off: int, v_off: int, ctx, q_out, k_pages, 
     nq, nk, nv = heads * head_dim, kv_heads * head_dim, kv_heads * v_head_dim
     if max(q_off + nq, k_off + nk, v_off + nv) > proj.shape[1] or tuple(q_out.shape) != (T, nq):
         raise KernelError(f"qk_norm_rope: proj {tuple(proj.shape)} against {nq} + {nk} + {nv} columns, q_out {tuple(q_out.shape)}")
-    for name, w, n in (("q_norm", q_norm, nq), ("k_norm", k_norm, nk)):
+    weighted = head_norm == "weighted"
+    for name, w, n in (("q_norm", q_norm, head_dim if weighted else nq), ("k_norm", k_norm, head_dim if weighted else nk)):
         if w is not None:
             _cuda(name, w, torch.float32)
             if w.numel() != n:
@@ -1048,7 +1093,9 @@ def qk_norm_rope(proj, q_off: int, k_off: int, v_off: int, ctx, q_out, k_pages, 
         _cuda("freq", freq, torch.float32)
         if rot_dims % 2 or rot_dims > head_dim or freq.numel() != rot_dims // 2:
             raise KernelError(f"qk_norm_rope: {rot_dims} rotated entries of {head_dim}, {freq.numel()} frequencies")
-    if head_norm and (q_norm is not None or k_norm is not None):
+    if weighted and (q_norm is None or k_norm is None):
+        raise KernelError("qk_norm_rope: the per-head norm before the rotation needs its weights")
+    if head_norm and not weighted and (q_norm is not None or k_norm is not None):
         raise KernelError("qk_norm_rope: the per-head norm takes no weights")
     for name, t in (("v_first", v_first), ("v_keep", v_keep)):
         if t is not None:
@@ -1073,7 +1120,7 @@ def qk_norm_rope(proj, q_off: int, k_off: int, v_off: int, ctx, q_out, k_pages, 
           k_norm.data_ptr() if k_norm is not None else None, float(eps), freq.data_ptr() if rot_dims else None,
           int(rot_dims), int(bool(interleaved)), ctx.positions.data_ptr(), q_out.data_ptr(), _rows("q_out", q_out),
           k_pages.data_ptr() if slot_mapping is not None else None, v_pages.data_ptr() if slot_mapping is not None else None,
-          int(dkp), slot_mapping.data_ptr() if slot_mapping is not None else None, int(ps), int(bool(head_norm)),
+          int(dkp), slot_mapping.data_ptr() if slot_mapping is not None else None, int(ps), 2 if weighted else int(bool(head_norm)),
           v_first.data_ptr() if v_first is not None else None, _rows("v_first", v_first) if v_first is not None else 0,
           v_lambda.data_ptr() if v_first is not None else None, v_keep.data_ptr() if v_keep is not None else None,
           _rows("v_keep", v_keep) if v_keep is not None else 0, T, _dt(proj), _stream())
@@ -1161,7 +1208,8 @@ def norm_scale_add(y, weight, scale, x, eps: float, *, pairs=None, pair_weights=
     """x += (v / sqrt(mean(v^2) + eps) * weight) * scale, row by row, all 32-bit; ``scale`` (a vector) may be None.
     v = y, plus sum_k pair_weights[t, k] * pairs[t * top + k] when ``pairs`` [T * top, D] is given (the chosen experts'
     results of a routed feed-forward; y may then be None).  With ``next_weight`` the new x is also normed for the branch
-    that reads it next: next_out = x / sqrt(mean(x^2) + next_eps) * (next_weight + next_offset), float32 or bfloat16."""
+    that reads it next: next_out = x / sqrt(mean(x^2) + next_eps) * (next_weight + next_offset), float32 or bfloat16;
+    with ``next_out`` alone the new x is copied there as it is."""
     _cuda("x", x, torch.float32, contiguous=False)
     _cuda("weight", weight, torch.float32)
     if scale is not None:
@@ -1182,15 +1230,18 @@ def norm_scale_add(y, weight, scale, x, eps: float, *, pairs=None, pair_weights=
         raise KernelError("norm_scale_add: nothing to add")
     if next_weight is not None:
         _cuda("next_weight", next_weight, torch.float32)
-        _cuda("next_out", next_out, contiguous=False)
-        if next_weight.numel() != D or tuple(next_out.shape) != (R, D):
+        if next_weight.numel() != D or next_out is None:
             raise KernelError("norm_scale_add: the next norm does not fit")
+    if next_out is not None:
+        _cuda("next_out", next_out, contiguous=False)
+        if tuple(next_out.shape) != (R, D):
+            raise KernelError("norm_scale_add: the next branch's input does not fit")
     _call("mllm_norm_scale_add", y.data_ptr() if y is not None else None, _rows("y", y) if y is not None else 0,
           pairs.data_ptr() if pairs is not None else None, pair_weights.data_ptr() if pairs is not None else None, int(top),
           weight.data_ptr(), scale.data_ptr() if scale is not None else None, x.data_ptr(), _rows("x", x),
           next_weight.data_ptr() if next_weight is not None else None, float(next_offset), float(next_eps),
-          next_out.data_ptr() if next_weight is not None else None, _rows("next_out", next_out) if next_weight is not None else 0,
-          R, D, float(eps), _dt(next_out) if next_weight is not None else F32, _stream())
+          next_out.data_ptr() if next_out is not None else None, _rows("next_out", next_out) if next_out is not None else 0,
+          R, D, float(eps), _dt(next_out) if next_out is not None else F32, _stream())
 
 
 def post_norm(x, weight, eps: float, alpha: float, *, y=None, pairs=None, pair_weights=None, top: int = 0, h=None) -> None:
@@ -1535,6 +1586,141 @@ def mlstm_step(proj, cols: dict, weight, state, ctx, out, *, heads: int, dim: in
           _dt(out), _stream())
 
 
+# --------------------------------------------------------------------------- retention
+RETENTION_MAX_DIM = 256      # most rows and columns of a head's state that csrc/retention.cu takes
+
+
+def _retention_sizes(name: str, proj, cols: dict, decay, state, heads: int, dim: int, vdim: int) -> None:
+    _cuda("proj", proj, torch.float32, contiguous=False)
+    _cuda("decay", decay, torch.float32)
+    _cuda("state", state, torch.float32)
+    width = {"q": heads * dim, "k": heads * dim, "v": heads * vdim, "g": heads * vdim}
+    for c, at in cols.items():
+        if at < 0 or at + width[c] > proj.shape[1]:
+            raise KernelError(f"{name}: columns of {c!r} at {at} in rows of {proj.shape[1]}")
+    if decay.numel() != heads:
+        raise KernelError(f"{name}: {decay.numel()} decays for {heads} heads")
+    if state.dim() != 2 or state.shape[1] < heads * dim * vdim:
+        raise KernelError(f"{name}: a state row of {state.shape[-1]} floats for {heads} heads of {dim} x {vdim}")
+
+
+def _freq_arg(name: str, freq, rot_dims: int, dim: int):
+    if rot_dims % 2 or rot_dims < 0 or rot_dims > dim:
+        raise KernelError(f"{name}: {rot_dims} rotated entries of {dim}")
+    if not rot_dims:
+        return None
+    _cuda("freq", freq, torch.float32)
+    if freq.numel() != rot_dims // 2:
+        raise KernelError(f"{name}: {freq.numel()} frequencies for {rot_dims} rotated entries")
+    return freq.data_ptr()
+
+
+def rotate_heads(proj, q_off: int, k_off: int, ctx, *, heads: int, dim: int, freq, rot_dims: int, interleaved: bool = False,
+                 k_scale: float = 1.0) -> None:
+    """In place on 32-bit proj [T, .]: the first ``rot_dims`` entries of every query head (at column q_off) and key head (at
+    k_off) turn by position * freq[i] (entry i pairs with i + rot_dims / 2, or 2i with 2i + 1 when ``interleaved``); all of a
+    key's entries are multiplied by ``k_scale``."""
+    _cuda("proj", proj, torch.float32, contiguous=False)
+    if min(q_off, k_off) < 0 or max(q_off, k_off) + heads * dim > proj.shape[1]:
+        raise KernelError(f"rotate_heads: {heads} heads of {dim} at columns {q_off} and {k_off} of {proj.shape[1]}")
+    _call("mllm_rotate_heads", proj.data_ptr(), _rows("proj", proj), int(q_off), int(k_off), heads, dim,
+          _freq_arg("rotate_heads", freq, rot_dims, dim), int(rot_dims), int(bool(interleaved)), float(k_scale),
+          ctx.positions.data_ptr(), proj.shape[0], _stream())
+
+
+def retention_scan(proj, cols: dict, decay, state, ctx, raw, *, heads: int, dim: int, vdim: int, write_state: bool = True,
+                   want_cols: int = 0) -> None:
+    """S <- decay_h S + k v^T, raw = S^T q over the step's tokens, request by request and head by head.  proj 32-bit [T, .] with
+    the columns ``cols`` = {"q", "k", "v"} -> first column (queries and keys already rotated); decay float32 [heads]; state
+    [slots, >= heads * dim * vdim]: S [heads, dim, vdim]; raw [T, heads * vdim] 32-bit."""
+    _retention_sizes("retention_scan", proj, {c: cols[c] for c in "qkv"}, decay, state, heads, dim, vdim)
+    _cuda("raw", raw, torch.float32)
+    if tuple(raw.shape) != (proj.shape[0], heads * vdim):
+        raise KernelError("retention_scan: raw does not fit")
+    _call("mllm_retention_scan", proj.data_ptr(), _rows("proj", proj), cols["q"], cols["k"], cols["v"], decay.data_ptr(),
+          state.data_ptr(), state.stride(0), ctx.cu_q.data_ptr(), ctx.state_slots.data_ptr(), raw.data_ptr(), ctx.S, heads, dim, vdim,
+          int(write_state), int(want_cols), _stream())
+
+
+def retention_finish(raw, proj, g_off: int, out, *, heads: int, vdim: int, eps: float) -> None:
+    """out = raw / sqrt(mean(raw^2) + eps) per head (no weight) * silu(g), g the heads * vdim columns of proj at ``g_off``."""
+    _cuda("raw", raw, torch.float32)
+    _cuda("proj", proj, torch.float32, contiguous=False)
+    _cuda("out", out, contiguous=False)
+    T = proj.shape[0]
+    if tuple(out.shape) != (T, heads * vdim) or tuple(raw.shape) != (T, heads * vdim) or g_off < 0 or g_off + heads * vdim > proj.shape[1]:
+        raise KernelError("retention_finish: shapes do not fit")
+    _call("mllm_retention_finish", raw.data_ptr(), proj.data_ptr(), _rows("proj", proj), int(g_off), out.data_ptr(), _rows("out", out), T,
+          heads, vdim, float(eps), _dt(out), _stream())
+
+
+def retention_step_ok(dim: int, vdim: int) -> bool:
+    """Whether the single-launch kernel takes steps of single tokens of these sizes."""
+    return library().mllm_retention_step_ok(dim, vdim) == 1
+
+
+def retention_step(proj, cols: dict, decay, state, ctx, out, *, heads: int, dim: int, vdim: int, freq, rot_dims: int,
+                   interleaved: bool = False, k_scale: float = 1.0, eps: float = 0.0, write_state: bool = True) -> None:
+    """``rotate_heads``, ``retention_scan`` and ``retention_finish`` of a step of single tokens in one launch (the same state
+    bit for bit); proj (queries and keys not yet rotated) is left as it is."""
+    _retention_sizes("retention_step", proj, cols, decay, state, heads, dim, vdim)
+    _cuda("out", out, contiguous=False)
+    if tuple(out.shape) != (proj.shape[0], heads * vdim) or proj.shape[0] != ctx.S:
+        raise KernelError("retention_step: shapes do not fit")
+    _call("mllm_retention_step", proj.data_ptr(), _rows("proj", proj), cols["q"], cols["k"], cols["v"], cols["g"], decay.data_ptr(),
+          _freq_arg("retention_step", freq, rot_dims, dim), int(rot_dims), int(bool(interleaved)), float(k_scale),
+          ctx.positions.data_ptr(), state.data_ptr(), state.stride(0), ctx.cu_q.data_ptr(), ctx.state_slots.data_ptr(), out.data_ptr(),
+          _rows("out", out), ctx.S, heads, dim, vdim, float(eps), int(write_state), _dt(out), _stream())
+
+
+# --------------------------------------------------------------------------- selective scan (a state per channel)
+SELECTIVE_MAX_STATE, SELECTIVE_MAX_RANK = 256, 10240     # what csrc/selective_scan.cu takes
+
+
+def _selective_sizes(name: str, x, bc, b_off, c_off, z, A, skip, dt_bias, state, out):
+    for k, t in (("x", x), ("bc", bc), ("z", z), ("out", out)):
+        _cuda(k, t, x.dtype, contiguous=False)
+    for k, t in (("A", A), ("skip", skip), ("dt_bias", dt_bias), ("state", state)):
+        _cuda(k, t, torch.float32)
+    T, C = x.shape
+    N = A.shape[1]
+    if A.shape[0] != C or skip.numel() != C or dt_bias.numel() != C or tuple(z.shape) != (T, C) or tuple(out.shape) != (T, C) \
+            or bc.shape[0] != T or min(b_off, c_off) < 0 or max(b_off, c_off) + N > bc.shape[1] or state.dim() != 2 \
+            or state.shape[1] < C * N or N > SELECTIVE_MAX_STATE:
+        raise KernelError(f"{name}: shapes do not fit")
+    return T, C, N
+
+
+def selective_scan(x, dt, bc, b_off: int, c_off: int, z, A, skip, dt_bias, state, ctx, out, *, out_scale: float = 1.0,
+                   write_state: bool = True) -> None:
+    """The selective scan with a state per channel over the step's tokens, request by request: d = softplus(dt + dt_bias);
+    S[c, n] <- exp(d_c A[c, n]) S[c, n] + d_c x_c B_n; out_c = out_scale * (sum_n S[c, n] C_n + skip_c x_c) * silu(z_c).
+    x, z, out [T, C] and bc [T, .] (B at column b_off, C at c_off) in one dtype; dt float32 [T, C]; A float32 [C, N] (negative);
+    state [slots, >= C * N]: S [C, N]."""
+    T, C, N = _selective_sizes("selective_scan", x, bc, b_off, c_off, z, A, skip, dt_bias, state, out)
+    _cuda("dt", dt, torch.float32, contiguous=False)
+    if tuple(dt.shape) != (T, C):
+        raise KernelError("selective_scan: one step size per token and channel")
+    _call("mllm_selective_scan", x.data_ptr(), _rows("x", x), dt.data_ptr(), _rows("dt", dt), bc.data_ptr(), _rows("bc", bc), int(b_off),
+          int(c_off), z.data_ptr(), _rows("z", z), A.data_ptr(), skip.data_ptr(), dt_bias.data_ptr(), state.data_ptr(), state.stride(0),
+          ctx.cu_q.data_ptr(), ctx.state_slots.data_ptr(), out.data_ptr(), _rows("out", out), ctx.S, C, N, float(out_scale),
+          int(write_state), _dt(x), _stream())
+
+
+def selective_step(x, low, rank: int, b_off: int, c_off: int, dt_weight, z, A, skip, dt_bias, state, ctx, out, *,
+                   out_scale: float = 1.0, write_state: bool = True) -> None:
+    """A step of single tokens: the step sizes' projection dt = dt_weight low[:, :rank] and ``selective_scan`` in one launch.
+    dt_weight [C, rank rounded up to 8] in x's dtype, zeros beyond the rank; low [T, .] also holds B and C."""
+    T, C, N = _selective_sizes("selective_step", x, low, b_off, c_off, z, A, skip, dt_bias, state, out)
+    _cuda("dt_weight", dt_weight, x.dtype)
+    if tuple(dt_weight.shape) != (C, -(-rank // 8) * 8) or rank > low.shape[1] or rank > SELECTIVE_MAX_RANK or T != ctx.S:
+        raise KernelError(f"selective_step: dt_weight {tuple(dt_weight.shape)} of rank {rank}")
+    _call("mllm_selective_step", x.data_ptr(), _rows("x", x), low.data_ptr(), _rows("low", low), int(rank), int(b_off), int(c_off),
+          dt_weight.data_ptr(), z.data_ptr(), _rows("z", z), A.data_ptr(), skip.data_ptr(), dt_bias.data_ptr(), state.data_ptr(),
+          state.stride(0), ctx.cu_q.data_ptr(), ctx.state_slots.data_ptr(), out.data_ptr(), _rows("out", out), ctx.S, C, N,
+          float(out_scale), int(write_state), _dt(x), _stream())
+
+
 # --------------------------------------------------------------------------- state-space mixer
 SSD_MAX_STATE_ROWS, SSD_MAX_TAPS = 256, 16       # what csrc/ssd.cu takes
 
@@ -1542,19 +1728,21 @@ SSD_MAX_STATE_ROWS, SSD_MAX_TAPS = 256, 16       # what csrc/ssd.cu takes
 def ssd_conv(proj, off: int, weight, bias, state, conv_off: int, ctx, out, *, write_state: bool = True) -> None:
     """out[t, c] = silu(bias[c] + sum_j weight[c, j] * u[t - (taps-1) + j, c]) with u = proj[:, off : off + C] within a
     request; inputs before the step's first token of a request come from state[slot, conv_off:] ([taps-1, C], oldest
-    first), which afterwards holds the request's last taps - 1 inputs.  out 32-bit [T, C]."""
+    first), which afterwards holds the request's last taps - 1 inputs.  out [T, C] 32-bit or in proj's dtype."""
     _cuda("proj", proj, contiguous=False)
     _cuda("weight", weight, torch.float32)
     _cuda("bias", bias, torch.float32)
     _cuda("state", state, torch.float32)
-    _cuda("out", out, torch.float32)
+    _cuda("out", out)
+    if out.dtype not in (torch.float32, proj.dtype):
+        raise KernelError(f"ssd_conv: out {out.dtype} for {proj.dtype} inputs")
     C, taps = weight.shape
     T = proj.shape[0]
     if tuple(out.shape) != (T, C) or bias.numel() != C or state.dim() != 2 or conv_off + (taps - 1) * C > state.shape[1]:
         raise KernelError("ssd_conv: shapes do not fit")
     _call("mllm_ssd_conv", proj.data_ptr(), _rows("proj", proj), int(off), weight.data_ptr(), bias.data_ptr(), state.data_ptr(),
           state.stride(0), int(conv_off), ctx.token_seq.data_ptr(), ctx.cu_q.data_ptr(), ctx.state_slots.data_ptr(),
-          out.data_ptr(), T, ctx.S, C, taps, int(write_state), _dt(proj), _stream())
+          out.data_ptr(), int(out.dtype == proj.dtype), T, ctx.S, C, taps, int(write_state), _dt(proj), _stream())
     if write_state and taps > 1 and T != ctx.S:
         global launches
         launches += 1       # the state's update (steps of single tokens do both in one launch)
@@ -1607,13 +1795,16 @@ _moe_few_tokens = None
 
 
 def moe_route(h, router, idx, weights, offsets, order, *, top: int, groups: int = 1, keep: int = 1, bias=None,
-              mode: str = "softmax_all", group_sum: int = 1, weight_scale: float = 1.0) -> None:
+              mode: str = "softmax_all", group_sum: int = 1, weight_scale: float = 1.0, correction=None, renorm: bool = True,
+              gate_weight=None, gate=None) -> None:
     """Per row of h: softmax of the router's logits (32-bit) over all experts; the best ``keep`` of ``groups`` equal
     groups of neighbours (by their largest score); the ``top`` best experts within them -> idx [T, top] (int32) and
     weights [T, top] (scores over their sum + 1e-20).  ``bias`` (float32 [E]) is added to the logits first.  ``mode``
     "softmax_top": the ``top`` largest logits are chosen and weighted by the softmax over those alone (no groups);
     "sigmoid": the scores are sigmoid(logit), expert by expert.  ``group_sum`` 2: a group's score is the sum of its two
-    largest scores.  The weights are multiplied by ``weight_scale``.
+    largest scores.  The weights are multiplied by ``weight_scale``.  ``correction`` (float32 [E]) is added to the scores
+    for the choice alone; ``renorm`` False: the weights are the chosen scores as they are.  ``gate_weight`` [1, D] (h's dtype)
+    with ``gate`` (float32 [T]): gate[t] = sigmoid(gate_weight . h[t]), for a shared expert that is gated.
     Then the (row, choice) pairs ordered by expert: offsets [E + 1], order [T * top]."""
     _cuda("h", h, contiguous=False)
     _cuda("router", router, h.dtype)
@@ -1629,11 +1820,22 @@ def moe_route(h, router, idx, weights, offsets, order, *, top: int, groups: int 
         _cuda("bias", bias, torch.float32)
         if bias.numel() != E:
             raise KernelError("moe_route: one bias per expert")
+    if correction is not None:
+        _cuda("correction", correction, torch.float32)
+        if correction.numel() != E:
+            raise KernelError("moe_route: one correction per expert")
+    if gate_weight is not None:
+        _cuda("gate_weight", gate_weight, h.dtype)
+        _cuda("gate", gate, torch.float32)
+        if gate_weight.numel() != D or gate.numel() != T:
+            raise KernelError("moe_route: the gate does not fit")
     modes = {"softmax_all": 0, "softmax_top": 1, "sigmoid": 2}
     if mode not in modes:
         raise KernelError(f"moe_route: unknown mode {mode!r}")
     _call("mllm_moe_route", h.data_ptr(), _rows("h", h), router.data_ptr(), bias.data_ptr() if bias is not None else None,
           modes[mode], T, D, E, int(top), int(groups), int(keep), int(group_sum), float(weight_scale),
+          correction.data_ptr() if correction is not None else None, int(bool(renorm)),
+          gate_weight.data_ptr() if gate_weight is not None else None, gate.data_ptr() if gate_weight is not None else None,
           idx.data_ptr(), weights.data_ptr(), offsets.data_ptr(), order.data_ptr(), _dt(h), _stream())
     global launches, _moe_few_tokens
     if _moe_few_tokens is None:
@@ -1643,12 +1845,14 @@ def moe_route(h, router, idx, weights, offsets, order, *, top: int, groups: int 
 
 
 def moe_grouped(a, weight, out, offsets, order, *, top: int, first: bool, act: str = "silu", limit: float = 0.0,
-                alpha: float = 1.0) -> None:
+                alpha: float = 1.0, identity: int = 0, self_rows=None) -> None:
     """The experts' products over the pairs in ``order``.  ``first``: a [T, K] (row = pair // top), weight [E, 2F, K]
     (gate rows, then up rows) -> out[i] = silu(gate) * up (``act`` "swiglu_clamp": the clamped form of gated_act, with
     ``limit`` and ``alpha``) for the i-th pair in order, [T*top, F]; ``act`` "relu_sq": experts without a gate, weight
     [E, F, K], out[i] = relu(.)^2.  Otherwise: a [T*top, K]
-    in that order, weight [E, N, K] -> out[pair] [T*top, N] 32-bit, by pair id."""
+    in that order, weight [E, N, K] -> out[pair] [T*top, N] 32-bit, by pair id.  The last ``identity`` of E + identity experts
+    have no weights and give their input back: the first product leaves their pairs out, the second copies the rows
+    (pair // top) of ``self_rows`` [T, N] (the tokens' inputs, in a's dtype)."""
     _cuda("a", a, contiguous=False)
     _cuda("weight", weight, a.dtype)
     _cuda("out", out, contiguous=False)
@@ -1656,8 +1860,14 @@ def moe_grouped(a, weight, out, offsets, order, *, top: int, first: bool, act: s
     n_pairs = order.numel()
     ungated = first and act in _UNGATED_ACT
     N = rows // 2 if (first and not ungated) else rows
-    if a.shape[1] != K or tuple(out.shape) != (n_pairs, N) or offsets.numel() != E + 1:
+    if a.shape[1] != K or tuple(out.shape) != (n_pairs, N) or offsets.numel() != E + identity + 1:
         raise KernelError("moe_grouped: shapes do not fit")
+    own = None
+    if identity and not first:
+        _cuda("self_rows", self_rows, a.dtype, contiguous=False)
+        if tuple(self_rows.shape) != (n_pairs // top, N):
+            raise KernelError(f"moe_grouped: self_rows {tuple(self_rows.shape)} for {n_pairs // top} tokens of {N}")
+        own = self_rows
     if act not in ("silu", "swiglu_clamp", *_UNGATED_ACT) or (act == "swiglu_clamp" and not limit > 0):
         raise KernelError(f"moe_grouped: activation {act!r} (limit {limit})")
     if (first and out.dtype != a.dtype) or (not first and out.dtype != torch.float32):
@@ -1665,6 +1875,7 @@ def moe_grouped(a, weight, out, offsets, order, *, top: int, first: bool, act: s
     _call("mllm_moe_grouped", a.data_ptr(), _rows("a", a), weight.data_ptr(), out.data_ptr(), _rows("out", out),
           offsets.data_ptr(), order.data_ptr(), n_pairs, E, N, K, int(top) if first else 0, 0 if first else 1,
           (2 if ungated else 0) if first else 1, _UNGATED_ACT[act] if ungated else _GATE_ACT[act], float(limit), float(alpha),
+          own.data_ptr() if own is not None else None, _rows("self_rows", own) if own is not None else 0, E + int(identity), int(top),
           _dt(a), _stream())
 
 

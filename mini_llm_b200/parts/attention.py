@@ -201,7 +201,11 @@ class RotaryAttention(ProjectedMixer):
     slope_h = 2^(-8 (h + 1) / H).  ``value_mix``: "first": the values of the step's tokens are also kept in a buffer of
     the step (``value_mix_key`` names it) for later layers; "mix": the values become (1 - lambda) v + lambda v_first
     before they are cached, v_first that buffer's rows of the same tokens and lambda a trained scalar (``v_mix``; a
-    "first" layer has the tensor too and does not use it).
+    "first" layer has the tensor too and does not use it).  ``head_norm`` "weighted": before the rotation every query head
+    and every key head is divided by its own root mean square and multiplied by a weight of head_dim entries, one for the
+    queries (q_norm) and one for the keys (k_norm).  ``keep_first`` f: the first f tokens stay visible beyond the window or
+    the block.  ``out_gate``: the joined heads are multiplied, entry by entry, with sigmoid(W_g h); W_g's rows stand behind
+    the values' in the input product.
 
     The keys are cached normed and rotated (rows padded to 16-byte pieces), so a cached token is never touched again.
     With a chunk mask the pages of finished blocks go back to the pool as the request moves on.
@@ -215,12 +219,17 @@ class RotaryAttention(ProjectedMixer):
                  rot_interleaved: bool = True, window: Optional[int] = None, chunk: Optional[int] = None, sink: bool = False,
                  head_norm: bool = False, rot_scaling: Optional[dict] = None, bias: bool = False,
                  softcap: Optional[float] = None, distance_slopes: bool = False, value_mix: Optional[str] = None,
-                 value_mix_key: str = "v_first"):
+                 value_mix_key: str = "v_first", keep_first: int = 0, out_gate: bool = False):
         self.hidden_size, self.num_heads, self.num_kv_heads = int(hidden_size), int(num_heads), int(num_kv_heads)
         self.head_dim, self.v_head_dim = int(head_dim), int(v_head_dim)
         self.scale, self.norm_eps = float(scale), float(norm_eps)
         self.qk_norm = bool(qk_norm)
-        self.head_norm = bool(head_norm)
+        self.head_norm = head_norm if head_norm == "weighted" else bool(head_norm)
+        self.keep_first, self.out_gate = int(keep_first), bool(out_gate)
+        if self.keep_first < 0:
+            raise ValueError(f"rotary attention: keep_first={keep_first}")
+        if self.out_gate:
+            self.in_names = ("q_weight", "k_weight", "v_weight", "g_weight")
         if self.qk_norm and self.head_norm:
             raise ValueError("rotary attention: a norm over the whole projection or one per head, not both")
         self.rot_scaling = None if rot_scaling is None else dict(rot_scaling)
@@ -262,6 +271,11 @@ class RotaryAttention(ProjectedMixer):
         if self.qk_norm:
             p["q_norm"] = ParamSpec((self.q_size,), "vector")
             p["k_norm"] = ParamSpec((self.k_size,), "vector")
+        if self.head_norm == "weighted":
+            p["q_norm"] = ParamSpec((self.head_dim,), "vector")
+            p["k_norm"] = ParamSpec((self.head_dim,), "vector")
+        if self.out_gate:
+            p["g_weight"] = ParamSpec((self.num_heads * self.v_head_dim, self.hidden_size), "matrix")
         if self.has_sink:
             p["sink"] = ParamSpec((self.num_heads,), "vector")
         return p
@@ -272,13 +286,15 @@ class RotaryAttention(ProjectedMixer):
             out.append(f"rotary attention: key size {self.head_dim} is not between 1 and 256")
         if not (1 <= self.v_head_dim <= 256):
             out.append(f"rotary attention: value size {self.v_head_dim} is not between 1 and 256")
-        if (self.q_size + self.k_size) * 4 * (2 if self.head_norm else 1) > 200 * 1024:
+        factors = self.rot_dims + self.num_heads + self.num_kv_heads
+        if ((self.q_size + self.k_size) * (2 if self.head_norm is True else 1) + factors) * 4 > 200 * 1024:
             out.append(f"rotary attention: a token's {self.q_size} + {self.k_size} query and key entries do not fit the "
                        f"shared memory of the kernel that norms and rotates them")
         return out
 
     def cache_need(self):
         return PagedNeed(kv_heads=self.num_kv_heads, head_dim=self.k_row, window=self.window, chunk=self.chunk,
+                         keep_first=self.keep_first if (self.window is not None or self.chunk is not None) else 0,
                          v_head_dim=None if self.v_head_dim == self.k_row else self.v_head_dim)
 
     def bind(self, params, rt) -> None:
@@ -291,7 +307,10 @@ class RotaryAttention(ProjectedMixer):
             f, _ = rotary_table(self.rot_dims, self.rot_base, self.rot_scaling)   # float64 -> float32; the kernel takes position * f in 32-bit
             self.freq = torch.tensor(f, dtype=torch.float64).float().contiguous().to(rt.device)
         if self.has_bias:
-            self.in_bias = torch.cat([self.q_bias, self.k_bias, self.v_bias]).contiguous()
+            parts = [self.q_bias, self.k_bias, self.v_bias]
+            if self.out_gate:
+                parts.append(torch.zeros_like(self.q_bias[:1]).expand(self.num_heads * self.v_head_dim))
+            self.in_bias = torch.cat(parts).contiguous()
         if self.distance_slopes:
             H = self.num_heads
             self.slopes = torch.tensor([2.0 ** (-8.0 * (h + 1) / H) for h in range(H)], dtype=torch.float64).float().to(rt.device)
@@ -316,7 +335,8 @@ class RotaryAttention(ProjectedMixer):
                          head_norm=self.head_norm, **mix)
         ops.biased_attention(q, cache.k_pages, cache.v_pages, gv.block_table, ctx, out, num_heads=self.num_heads,
                              num_kv_heads=self.num_kv_heads, scale=self.scale, out_scale=out_scale, window=self.window,
-                             chunk=self.chunk, sink=self.sink, softcap=self.softcap or 0.0, slopes=self.slopes)
+                             chunk=self.chunk, sink=self.sink, softcap=self.softcap or 0.0, slopes=self.slopes,
+                             keep_first=self.keep_first, gate=proj[:, self.q_size + self.k_size + self.v_size:] if self.out_gate else None)
 
 
 register_part("mixer", "rotary_attention", RotaryAttention)

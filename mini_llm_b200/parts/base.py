@@ -23,6 +23,9 @@ Interfaces (all tensors are CUDA tensors on the engine's stream):
 * Head:          ``forward(y[R,D], ctx) -> logits_f32[R,V]``.
 * PassInput:     ``forward(x_f32[T,D], x0_f32[T,D], ctx, t) -> x``: makes the residual anew at the start of pass t of a
                  looped stretch of layers, from what it was and the embedded rows x0.
+* TokenTable:    a table with a row per token of the vocabulary that every layer may read a part of (``table``).
+* TokenSide:     ``forward(h[T,D], ctx, y_f32[T,D])``: writes a layer's branch that depends on the token itself (its part of
+                 the model's ``TokenTable``, taken by ``attach``) and on h.
 * Join:          ``forward(y_f32[T,D], x_f32[T,D], ctx)``: brings a branch's result y into the residual x
                  (a norm and a scale on y, say).  Mixers and feed-forwards with ``can_overwrite = True``
                  take ``accumulate=False`` and then write their result instead of adding it.
@@ -103,6 +106,20 @@ class PassInput(Part):
         raise NotImplementedError
 
 
+class TokenTable(Part):
+    category = "token_table"
+
+
+class TokenSide(Part):
+    category = "token_side"
+
+    def attach(self, table) -> None:
+        self.source = table
+
+    def forward(self, h, ctx, y):  # pragma: no cover
+        raise NotImplementedError
+
+
 class Positions(Part):
     category = "positions"
     max_positions: Optional[int] = None
@@ -131,7 +148,7 @@ class Head(Part):
 
 _REGISTRIES: Dict[str, Dict[str, Callable[..., Any]]] = {
     "norm": {}, "mixer": {}, "feed_forward": {}, "positions": {}, "embedding": {}, "head": {},
-    "arrangement": {}, "join": {}, "pass_input": {},
+    "arrangement": {}, "join": {}, "pass_input": {}, "token_table": {}, "token_side": {},
 }
 
 

@@ -7,6 +7,9 @@ x += mixer(norm(x)); x += ff(norm(x)), with the residual stream x in 32-bit.
 join (a second norm and a scale per column, say) before it reaches x.
 "post_norm": x = norm_a(alpha * x + mixer(x)); x = norm_b(alpha * x + ff(x)): the branches read x itself and the norm
 comes after the sum (the joins are ``parts.join.PostNormJoin``); the layer has no norms in front of its branches.
+"output_norm": x = x + m * norm_a(mixer(x)); x = x + m * norm_b(ff(x)): the branches read x itself and only their results
+are normed (the joins are ``parts.join.NormScaleJoin``).
+In "output_norm" a layer may also have a third branch, ``LayerSpec.side``, an input of the token of its own.
 """
 from __future__ import annotations
 
@@ -136,8 +139,36 @@ def _take_act_copy(ctx, x, act_dtype):
         return left[2]
     if x.dtype == act_dtype:
         return x
-    raise RuntimeError("post_norm arrangement: nobody left a copy of the residual in the activation dtype "
-                       "(the embedding of such a model norms its rows and leaves one)")
+    raise RuntimeError("nobody left a copy of the residual in the activation dtype (the embedding of a model whose layers "
+                       "read it leaves one)")
 
 
 register_part("arrangement", "post_norm", lambda: post_norm)
+
+
+def output_norm(layer, x, ctx, cache):
+    """x <- x + n(branch(x)) for the mixer, the feed-forward (if there is one) and the token's own input to the layer (if there
+    is one), n the branch's join: a norm of the branch's result with a constant.  A branch reads x as the products take it;
+    the join before it left that copy."""
+    import torch
+    if layer.mixer_join is None or (layer.ff is not None and layer.ff_join is None) or (layer.side is not None and layer.side_join is None):
+        raise RuntimeError("output_norm arrangement: the layer has no join for a branch")
+    h = _take_act_copy(ctx, x, layer.mixer.rt.act_dtype)
+    y = ctx.ws.buf("branch_out", x.shape[0], x.shape[1], torch.float32)
+    _branch(layer.mixer, y, h, ctx, cache)
+    h = layer.mixer_join.forward(y, x, ctx, then_copy=True)
+    if layer.ff is not None:
+        if hasattr(layer.ff, "forward_pairs") and getattr(layer.ff_join, "takes_pairs", False):
+            shared, pairs = layer.ff.forward_pairs(h, ctx, y)
+            h = layer.ff_join.forward(y if shared else None, x, ctx, pairs=pairs, then_copy=True)
+        else:
+            _branch(layer.ff, y, h, ctx)
+            h = layer.ff_join.forward(y, x, ctx, then_copy=True)
+    if layer.side is not None:
+        layer.side.forward(h, ctx, y)
+        h = layer.side_join.forward(y, x, ctx, then_copy=True)
+    leave_act_copy(ctx, x, h)
+    return x
+
+
+register_part("arrangement", "output_norm", lambda: output_norm)

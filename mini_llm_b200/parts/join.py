@@ -34,10 +34,13 @@ class NormScaleJoin(Join):
         if "weight" in params and self.factor != 1.0:       # the constant rides in the norm's weights
             self.weight = (self.weight * self.factor).contiguous()
 
-    def forward(self, y, x, ctx, pairs=None, then_norm=None):
+    def forward(self, y, x, ctx, pairs=None, then_norm=None, then_copy: bool = False):
         """x += n(y [+ the weighted pairs], w) * s.  ``pairs``: (results [T * top, D], weights [T, top], top) of a routed
         feed-forward whose weighted sum has not been taken yet (y may then be None).  ``then_norm``: an RMS norm that the
-        next branch applies to the new x; its result comes back (one kernel does both), else None."""
+        next branch applies to the new x; its result comes back (one kernel does both), else None.  ``then_copy``: the next
+        branch reads the new x as it is; it comes back as the products take it (x itself on the 32-bit path, a copy in the
+        activation dtype otherwise)."""
+        import torch
         ops = self.rt.ops
         kw = {}
         if pairs is not None:
@@ -47,6 +50,11 @@ class NormScaleJoin(Join):
             h = ctx.ws.buf("norm_out", x.shape[0], self.hidden_size, self.rt.act_dtype)
             kw.update(next_weight=then_norm.weight, next_eps=then_norm.eps, next_offset=1.0 if then_norm.unit_offset else 0.0,
                       next_out=h)
+        elif then_copy:
+            h = x
+            if self.rt.act_dtype != torch.float32:
+                h = ctx.ws.buf("act_copy", x.shape[0], self.hidden_size, self.rt.act_dtype)
+                kw.update(next_out=h)
         ops.norm_scale_add(y, self.weight, self.scale, x, self.eps, **kw)
         return h
 

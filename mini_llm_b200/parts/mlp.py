@@ -14,6 +14,7 @@ ACTIVATIONS = ("gelu_tanh", "gelu_erf")
 
 class MLP(FeedForward):
     accepts_lazy_norm = True
+    can_overwrite = True                # forward(..., accumulate=False) writes the result instead of adding it
 
     def __init__(self, hidden_size: int, inner_size: int, activation: str, bias: bool = True):
         if activation not in ACTIVATIONS:
@@ -33,11 +34,11 @@ class MLP(FeedForward):
             p["proj_bias"] = ParamSpec((self.hidden_size,), "vector")
         return p
 
-    def forward(self, h, ctx, out_accum):
+    def forward(self, h, ctx, out_accum, accumulate: bool = True):
         ops = self.rt.ops
         mid = ctx.ws.buf("ff_mid", h.shape[0], self.inner_size, self.rt.act_dtype)
         ops.linear(h, self.fc_weight, self.fc_bias, out=mid, act=self.activation)
-        ops.linear(mid, self.proj_weight, self.proj_bias, out=out_accum, accumulate=True)
+        ops.linear(mid, self.proj_weight, self.proj_bias, out=out_accum, accumulate=accumulate)
 
 
 register_part("feed_forward", "mlp", MLP)

@@ -42,6 +42,8 @@ class Layer:
         self.ff = build_part("feed_forward", spec.ff) if spec.ff is not None else None
         self.mixer_join = build_part("join", spec.mixer_join) if spec.mixer_join is not None else None
         self.ff_join = build_part("join", spec.ff_join) if (spec.ff is not None and spec.ff_join is not None) else None
+        self.side = build_part("token_side", spec.side) if spec.side is not None else None
+        self.side_join = build_part("join", spec.side_join) if (spec.side is not None and spec.side_join is not None) else None
         self.arrangement = get_part_factory("arrangement", spec.arrangement)()
 
 
@@ -51,6 +53,7 @@ class Model:
         self.embedding = build_part("embedding", spec.embedding)
         self.positions = build_part("positions", spec.positions)
         self.pass_input = build_part("pass_input", spec.pass_input) if spec.pass_input is not None else None
+        self.token_table = build_part("token_table", spec.token_table) if spec.token_table is not None else None
         self.layers: List[Layer] = [Layer(ls, spec.hidden_size) for ls in spec.layers]
         self.final_norm = build_part("norm", spec.final_norm)
         self.head = build_part("head", spec.head)
@@ -89,6 +92,9 @@ class Model:
         self.rt = rt
         if hasattr(self.head, "tie"):
             self.head.tie(self.embedding)
+        for l in self.layers:
+            if l.side is not None:
+                l.side.attach(self.token_table)
 
     def layer_cache(self, cache_manager, entry) -> LayerCache:
         owner = entry.cache_unit

@@ -67,6 +67,8 @@ class ParallelMixer(Mixer):
     ``scales``: the factor on each branch's result.  Parameters are named "<branch name>.<local name>"."""
 
     accepts_lazy_norm = True
+    can_overwrite = True                # forward(..., accumulate=False) writes the result instead of adding it
+    in_bias = None
 
     def __init__(self, branches: List[Dict[str, Any]], scales: Sequence[float]):
         if len(branches) != len(scales) or not branches:
@@ -103,6 +105,12 @@ class ParallelMixer(Mixer):
         if params:
             self.in_weight = torch.cat([b.in_weight for b in self.branches], 0).contiguous()
             self.out_weight = torch.cat([getattr(b, b.out_name) for b in self.branches], 1).contiguous()
+            if any(b.out_bias is not None or b.proj_f32 for b in self.branches):
+                raise ValueError("ParallelMixer: a branch has an output bias or wants its columns in 32-bit")
+            if any(b.in_bias is not None for b in self.branches):       # the branches' biases side by side, zeros where there is none
+                self.in_bias = torch.cat([b.in_bias if b.in_bias is not None else
+                                          torch.zeros(b.in_width, dtype=torch.float32, device=self.in_weight.device)
+                                          for b in self.branches]).contiguous()
             # the branches keep views of the joined matrices, not copies of their own
             r = c = 0
             for b in self.branches:
@@ -114,19 +122,20 @@ class ParallelMixer(Mixer):
                 setattr(b, b.out_name, self.out_weight[:, c:c + b.core_width])
                 c += b.core_width
 
-    def forward(self, h, ctx, cache, out_accum):
+    def forward(self, h, ctx, cache, out_accum, accumulate: bool = True):
         ops = self.rt.ops
         T = h.shape[0]
         n_in = self.in_weight.shape[0]
         proj = ctx.ws.buf("mix_proj", T, -(-n_in // 8) * 8, self.rt.act_dtype)[:, :n_in]    # rows stay 16-byte aligned
-        ops.linear(h, self.in_weight, None, out=proj)
-        mid = ctx.ws.buf("mix_core", T, self.out_weight.shape[1], self.rt.act_dtype)
+        ops.linear(h, self.in_weight, self.in_bias, out=proj)
+        wide = self.out_weight.shape[1]
+        mid = ctx.ws.buf("mix_core", T, -(-wide // 8) * 8, self.rt.act_dtype)[:, :wide]
         r = c = 0
         for b, s in zip(self.branches, self.scales):
             b.core(proj[:, r:r + b.in_width], ctx, cache, mid[:, c:c + b.core_width], out_scale=s)
             r += b.in_width
             c += b.core_width
-        ops.linear(mid, self.out_weight, None, out=out_accum, accumulate=True)
+        ops.linear(mid, self.out_weight, None, out=out_accum, accumulate=accumulate)
 
 
 register_part("mixer", "parallel", ParallelMixer)

@@ -14,6 +14,8 @@ Scaling by wavelength (``scaling`` = {factor, low, high, original}; the form Lla
 l_i = 2 pi / f_i is shorter than original / high keeps its frequency, one longer than original / low turns ``factor``
 times slower, and between the two the frequency is (1 - s) f_i / factor + s f_i with s = (original / l_i - low) /
 (high - low); cos and sin keep their size.
+
+Linear scaling (``scaling`` = {factor} alone): every frequency is divided by the factor; cos and sin keep their size.
 """
 from __future__ import annotations
 
@@ -29,6 +31,11 @@ def rotary_table(dims: int, base: float, scaling: Optional[dict] = None) -> Tupl
     f = [float(base) ** (-2.0 * i / dims) for i in range(half)]
     if not scaling:
         return f, 1.0
+    if set(scaling) == {"factor"}:
+        factor = float(scaling["factor"])
+        if not factor > 0:
+            raise ValueError(f"rotary: linear scaling needs a positive factor, got {scaling!r}")
+        return [fi / factor for fi in f], 1.0
     factor, orig = float(scaling["factor"]), float(scaling["original"])
     if "low" in scaling or "high" in scaling:
         low, high = float(scaling["low"]), float(scaling["high"])

@@ -63,6 +63,8 @@ class LayerSpec:
     arrangement: str = "pre_norm"
     mixer_join: Optional[PartSpec] = None
     ff_join: Optional[PartSpec] = None
+    side: Optional[PartSpec] = None          # category "token_side": a third branch that reads the token itself
+    side_join: Optional[PartSpec] = None
 
 
 @dataclass
@@ -100,6 +102,7 @@ class ModelSpec:
     final_norm: PartSpec
     head: PartSpec
     schedule: Optional[List[ScheduleEntry]] = None
+    token_table: Optional[PartSpec] = None   # category "token_table": what the layers' ``side`` branches read of a token
     pass_input: Optional[PartSpec] = None    # category "pass_input": runs before every entry that enters a pass
     max_positions: Optional[int] = None      # None: the position encoding sets no limit
     eos_token_id: Optional[int] = None
@@ -111,6 +114,8 @@ class ModelSpec:
         n = len(self.layers)
         if self.pass_input is None and any(e.enters_pass is not None for e in self.schedule):
             raise ValueError("the schedule enters a pass but the model names no pass_input part")
+        if self.token_table is None and any(l.side is not None for l in self.layers):
+            raise ValueError("a layer has a side branch but the model names no token_table part")
         private = 0
         for e in self.schedule:
             if not (0 <= e.layer < n) or not (0 <= e.cache_of < n):
@@ -125,6 +130,8 @@ class ModelSpec:
         """(label, PartSpec) of every part, in a fixed order."""
         yield "embedding", self.embedding
         yield "positions", self.positions
+        if self.token_table is not None:
+            yield "token_table", self.token_table
         if self.pass_input is not None:
             yield "pass_input", self.pass_input
         for i, l in enumerate(self.layers):
@@ -139,5 +146,9 @@ class ModelSpec:
                 yield f"layers.{i}.ff", l.ff
                 if l.ff_join is not None:
                     yield f"layers.{i}.ff_join", l.ff_join
+            if l.side is not None:
+                yield f"layers.{i}.side", l.side
+                if l.side_join is not None:
+                    yield f"layers.{i}.side_join", l.side_join
         yield "final_norm", self.final_norm
         yield "head", self.head

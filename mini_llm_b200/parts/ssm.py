@@ -1,4 +1,4 @@
-"""State-space mixers: a fixed-size state per request, carried from token to token.
+"""State-space mixers: a fixed-size state per request, carried from token to token (``MambaMixer``: see the class).
 
 ``Mamba2Mixer`` (state-space duality).  With inner = heads * vdim, N state rows and G groups, W_in h is
 [z: inner | x: inner | B: G*N | C: G*N | dt: heads].  x, B and C pass a causal convolution per channel (weights
@@ -77,3 +77,84 @@ class Mamba2Mixer(ProjectedMixer):
 
 
 register_part("mixer", "mamba2", Mamba2Mixer)
+
+
+class MambaMixer(ProjectedMixer):
+    """The selective scan with a state per channel (Mamba's first form).  W_in h is [x: inner | z: inner]; x passes the causal
+    convolution per channel (weights [inner, taps], a bias) and silu; W_x x is [dt: rank | B: N | C: N];
+    dt <- softplus(W_dt dt + bias), one per channel; A = -exp(A_log) [inner, N].  Per channel c, S zero at the start:
+
+        S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n        y_c = sum_n S[c, n] C_n + D_c x_c
+
+    and W_o (y * silu(z)).  The request's state holds S and the last taps - 1 inputs of the convolution, both 32-bit, in one
+    row of the cache manager's state arena; dt, the decays, the recurrence and the gate are 32-bit whatever the engine's
+    dtype."""
+
+    in_names = ("in_proj",)
+    out_name = "out_weight"
+
+    def __init__(self, hidden_size: int, inner: int, state_size: int, dt_rank: int, conv_taps: int):
+        self.hidden_size, self.inner, self.state_size = int(hidden_size), int(inner), int(state_size)
+        self.dt_rank, self.conv_taps = int(dt_rank), int(conv_taps)
+        self.ssm_floats = self.inner * self.state_size
+        self.state_floats = self.ssm_floats + (self.conv_taps - 1) * self.inner
+
+    def param_specs(self):
+        I, N, R = self.inner, self.state_size, self.dt_rank
+        return {"in_proj": ParamSpec((2 * I, self.hidden_size), "matrix"),
+                "conv_weight": ParamSpec((I, self.conv_taps), "vector"), "conv_bias": ParamSpec((I,), "vector"),
+                "x_proj": ParamSpec((R + 2 * N, I), "matrix"),
+                "dt_weight": ParamSpec((I, R), "matrix"), "dt_bias": ParamSpec((I,), "vector"),
+                "A_log": ParamSpec((I, N), "vector"), "D": ParamSpec((I,), "vector"),
+                "out_weight": ParamSpec((self.hidden_size, I), "matrix")}
+
+    def kernel_limits(self, dtype: str):
+        from .. import ops
+        out = []
+        if not (1 <= self.state_size <= ops.SELECTIVE_MAX_STATE):
+            out.append(f"mamba: a state of {self.state_size} entries per channel; the kernels take {ops.SELECTIVE_MAX_STATE}")
+        if not (1 <= self.dt_rank <= ops.SELECTIVE_MAX_RANK):
+            out.append(f"mamba: step sizes of rank {self.dt_rank}; the kernels take {ops.SELECTIVE_MAX_RANK}")
+        if not (1 <= self.conv_taps <= ops.SSD_MAX_TAPS):
+            out.append(f"mamba: a convolution of {self.conv_taps} taps; the kernel takes 1 to {ops.SSD_MAX_TAPS}")
+        return out
+
+    def cache_need(self):
+        return StateNeed((self.state_floats,), "float32")
+
+    def bind(self, params, rt) -> None:
+        import torch
+        super().bind(params, rt)
+        if "A_log" in params:
+            self.A = (-torch.exp(self.A_log.double())).float().contiguous()
+            # rows of the step sizes' projection padded to 16-byte pieces; the padding is zero
+            R8 = -(-self.dt_rank // 8) * 8
+            padded = torch.zeros((self.inner, R8), dtype=self.dt_weight.dtype, device=self.dt_weight.device)
+            padded[:, :self.dt_rank] = self.dt_weight
+            self.dt_narrow = self.dt_weight         # as stored, for tables too narrow for the padded columns
+            self.dt_weight = padded
+
+    def core(self, proj, ctx, cache, out, out_scale: float = 1.0) -> None:
+        import torch
+        ops = self.rt.ops
+        T, I, N, R = proj.shape[0], self.inner, self.state_size, self.dt_rank
+        R8, wide = self.dt_weight.shape[1], R + 2 * N
+        act = self.rt.act_dtype
+        x = ctx.ws.buf("mamba_x", T, -(-I // 8) * 8, act)[:, :I]
+        ops.ssd_conv(proj, 0, self.conv_weight, self.conv_bias, cache.state, self.ssm_floats, ctx, x, write_state=cache.write)
+        low = ctx.ws.buf("mamba_low", T, max(R8, -(-wide // 8) * 8), act)     # rows stay 16-byte aligned
+        ops.linear(x, self.x_proj, None, out=low[:, :wide])
+        z = proj[:, I:2 * I]
+        args = (z, self.A, self.D, self.dt_bias, cache.state, ctx, out)
+        if getattr(ctx, "decode_only", False):
+            ops.selective_step(x, low[:, :wide], R, R, R + N, self.dt_weight, *args, out_scale=out_scale, write_state=cache.write)
+            return
+        dt = ctx.ws.buf("mamba_dt", T, I, torch.float32)
+        if R8 <= wide:          # the columns beyond the rank are B's: finite, and their weights are zero
+            ops.linear(low[:, :R8], self.dt_weight, None, out=dt)
+        else:
+            ops.linear(low[:, :R], self.dt_narrow, None, out=dt)
+        ops.selective_scan(x, dt, low, R, R + N, *args, out_scale=out_scale, write_state=cache.write)
+
+
+register_part("mixer", "mamba", MambaMixer)
