@@ -40,7 +40,7 @@ with "impl": "reference" and "dtype": "fp32".  The reference holds at most 16 re
 (more are cut) and there is no batch-64 point.  Where it cannot be built or run the line is
 {"impl": "reference", "unavailable": "<why>"}.
 
-``--compare-designs [small,medium,large]`` measures the engine's other designs, Finuvik, Falisun, Mumopel, Kusirax and Zadenex,
+``--compare-designs [small,medium,large]`` measures the engine's other designs, Finuvik, Falisun, Mumopel, Kusirax, Zadenex and Zanelorn,
 beside GPT-2 at equal width, depth and head count (bfloat16 unless --dtype is given; ``--designs gpt2,falisun`` picks some).
 
 ``--profile-step prefill|decode [--kernel-times]`` runs one small eager step (for a profiler, or to
@@ -316,7 +316,7 @@ def profile_step(kind: str, dtype: str, layers: int, batch: int, kernel_times: b
     from mini_llm_b200.engine.runner import ModelRunner, StepEntry
 
     cfg = dict(SMALL, n_layer=layers)
-    if design in ("finuvik", "falisun", "mumopel", "kusirax", "zadenex"):  # the same step of the other designs at the "small" comparison size
+    if design in ("finuvik", "falisun", "mumopel", "kusirax", "zadenex", "zanelorn"):  # the same step of the other designs at the "small" comparison size
         cfg = design_configs("small")[design]
         cfg["layers"] = cfg["layers"][:layers]
         if cfg.get("loop") and cfg["loop"]["stop"] > layers:
@@ -522,7 +522,28 @@ def design_configs(size: str):
         zl.append(dict(type=kind, mixer=mixer, mlp=dict(kind="dense", ff=F)))
     zadenex = dict(architecture="Zadenex", width=D, vocab=DESIGN_VOCAB, norm=dict(eps=1e-5), embedding=dict(scale=4.0),
                    residual_mult=0.5, loop=dict(start=1, stop=2, times=1), layers=zl)
-    return {"gpt2": gpt2, "finuvik": finuvik, "falisun": falisun, "mumopel": mumopel, "kusirax": kusirax, "zadenex": zadenex}
+    # Zanelorn at the same width, heads and key/value heads: retention (heads of 64 x 64 over the whole width, as Zadenex's
+    # memory and Kusirax's recurrence; every entry turns) alternates with parallel layers (rotary attention over the last 768
+    # tokens and the first 4, beside a selective scan over as many channels as the width has columns, 16 entries each, step
+    # sizes of rank D/16); a dense feed-forward of Finuvik's inner size alternates with Mumopel's routed one (2 of 8 clamped
+    # experts, here beside 2 identity outputs and a gated shared expert); D/8 columns of the token's own row per layer
+    zr = dict(kind="moe", router=dict(experts=8, identity=2, top=2), expert=dict(ff=F // 4 // 8 * 8, limit=7.0),
+              shared=dict(ff=F // 2 // 8 * 8, limit=7.0))
+    nl = []
+    for i in range(L):
+        if i % 2 == 0:
+            n = D // 64
+            mixer = dict(heads=n, dim=64, vdim=64, decay=[1.0 - 2.0 ** -(5.0 + 4.0 * h / n) for h in range(n)],
+                         rot=dict(base=10000.0, dims=64))
+        else:
+            mixer = dict(left=dict(heads=H, kv_heads=z["kv_heads"], dim=dh, vdim=dh, scale=dh ** -0.5, mask=dict(size=768, keep_first=4),
+                                   rot=dict(base=10000.0, dims=dh, scaling=dict(factor=2.0))), left_scale=0.7,
+                         right=dict(inner=D, state=16, dt_rank=D // 16, conv=4), right_scale=0.7)
+        nl.append(dict(type="retention" if i % 2 == 0 else "parallel", mixer=mixer, mlp=dict(kind="dense", ff=F) if i % 2 == 0 else zr))
+    zanelorn = dict(architecture="Zanelorn", width=D, vocab=DESIGN_VOCAB, norm=dict(eps=1e-5), embedding=dict(scale=4.0),
+                    residual_mult=0.5, token_side=dict(dim=D // 8), layers=nl)
+    return {"gpt2": gpt2, "finuvik": finuvik, "falisun": falisun, "mumopel": mumopel, "kusirax": kusirax, "zadenex": zadenex,
+            "zanelorn": zanelorn}
 
 
 def _design_model(model_dir, dtype, batch, tokens):
@@ -785,7 +806,7 @@ def main() -> int:
     ap.add_argument("--no-points", action="store_true", help="skip the batch 1 / 64, prefill and other-precision measurements")
     ap.add_argument("--profile-step", choices=["prefill", "decode"],
                     help="run one small eager step for a profiler instead of the benchmark")
-    ap.add_argument("--design", choices=["gpt2", "finuvik", "falisun", "mumopel", "kusirax", "zadenex"], default="gpt2",
+    ap.add_argument("--design", choices=["gpt2", "finuvik", "falisun", "mumopel", "kusirax", "zadenex", "zanelorn"], default="gpt2",
                     help="with --profile-step: the model whose step is run (the other designs: the 'small' size of --compare-designs)")
     ap.add_argument("--kernel-times", action="store_true",
                     help="with --profile-step: time every launch of one eager step with CUDA events and print the shares")
@@ -796,7 +817,7 @@ def main() -> int:
     ap.add_argument("--compare-designs", nargs="?", const="small,medium,large", metavar="SIZES",
                     help="measure Finuvik, Falisun and Mumopel beside GPT-2 at equal sizes (a comma list of small, medium, large) "
                          "instead of the benchmark: prefill of 2 x 1024 tokens and decode at --batch, one JSON line per size")
-    ap.add_argument("--designs", default="", help="with --compare-designs: a comma list of gpt2, finuvik, falisun, mumopel, kusirax, zadenex (default: all)")
+    ap.add_argument("--designs", default="", help="with --compare-designs: a comma list of gpt2, finuvik, falisun, mumopel, kusirax, zadenex, zanelorn (default: all)")
     args = ap.parse_args()
     if args.compare_designs:
         sizes = [z for z in args.compare_designs.split(",") if z]

@@ -127,3 +127,69 @@ MLLM_EXPORT int mllm_token_side_gate(const float* z, long long ldz, const int* i
         return mllm_fail(1, "token_side_gate: unknown dtype code %d", dtype);
     return 0;
 }
+
+// Few tokens (decode steps): the gate's product and what token_side_gate makes of it in one launch.  grid (tokens, column
+// blocks of 8 * COLS), 8 warps: the token's row of h is staged in shared memory as 32-bit, a warp owns COLS columns and its
+// lanes split the sum, with 16-byte loads of the weight rows where they allow it.
+template <typename T, int COLS>
+__global__ void __launch_bounds__(256)
+token_side_mid_kernel(const T* h, long long ldh, const T* __restrict__ W, int D, const int* __restrict__ ids, const T* __restrict__ table,
+                      long long ldt, int off, T* __restrict__ out, long long ldo, int d) {
+    extern __shared__ float hs[];           // [D]
+    constexpr int V = 16 / sizeof(T);
+    const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int c0 = (blockIdx.y * 8 + warp) * COLS;
+    const T* row = table + (size_t)ids[t] * ldt + off;
+    pdl_wait();
+    pdl_launch();
+    for (int k = threadIdx.x; k < D; k += 256) hs[k] = to_f32(h[(size_t)t * ldh + k]);
+    __syncthreads();
+    if (c0 >= d) return;
+    float acc[COLS];
+#pragma unroll
+    for (int u = 0; u < COLS; ++u) acc[u] = 0.f;
+    if (D % V == 0 && (uintptr_t)W % 16 == 0) {
+#pragma unroll 2
+        for (int k = lane * V; k < D; k += 32 * V) {
+            uint4 w[COLS];
+#pragma unroll
+            for (int u = 0; u < COLS; ++u) w[u] = *reinterpret_cast<const uint4*>(W + (size_t)min(c0 + u, d - 1) * D + k);
+#pragma unroll
+            for (int u = 0; u < COLS; ++u) {
+                const T* p = reinterpret_cast<const T*>(&w[u]);
+#pragma unroll
+                for (int e = 0; e < V; ++e) acc[u] = fmaf(hs[k + e], to_f32(p[e]), acc[u]);
+            }
+        }
+    } else {
+        for (int k = lane; k < D; k += 32) {
+#pragma unroll
+            for (int u = 0; u < COLS; ++u) acc[u] = fmaf(hs[k], to_f32(W[(size_t)min(c0 + u, d - 1) * D + k]), acc[u]);
+        }
+    }
+#pragma unroll
+    for (int u = 0; u < COLS; ++u) {
+        const float v = warp_sum(acc[u]);
+        if (lane == 0 && c0 + u < d) out[(size_t)t * ldo + c0 + u] = from_f32<T>(gelu_tanh_f(v) * to_f32(row[c0 + u]));
+    }
+}
+
+MLLM_EXPORT int mllm_token_side_mid(const void* h, long long ldh, const void* W, int D, const int* ids, const void* table, long long ldt,
+                                    int off, void* out, long long ldo, int T, int d, int dtype, cudaStream_t stream) {
+    if (T <= 0) return 0;
+    if (d <= 0 || off < 0 || off + d > ldt) return mllm_fail(1, "token_side_mid: columns %d to %d of rows of %lld", off, off + d, ldt);
+    if (D <= 0 || (size_t)D * 4 > 48 * 1024) return mllm_fail(1, "token_side_mid: rows of %d", D);
+    constexpr int COLS = 2;
+    const dim3 grid(T, (d + 8 * COLS - 1) / (8 * COLS));
+    if (grid.y > 65535) return mllm_fail(1, "token_side_mid: %d columns", d);
+    if (dtype == MLLM_F32)
+        MLLM_CUDA(mllm_launch(token_side_mid_kernel<float, COLS>, grid, dim3(256), (size_t)D * 4, stream, true, (const float*)h, ldh,
+                              (const float*)W, D, ids, (const float*)table, ldt, off, (float*)out, ldo, d));
+    else if (dtype == MLLM_BF16)
+        MLLM_CUDA(mllm_launch(token_side_mid_kernel<__nv_bfloat16, COLS>, grid, dim3(256), (size_t)D * 4, stream, true,
+                              (const __nv_bfloat16*)h, ldh, (const __nv_bfloat16*)W, D, ids, (const __nv_bfloat16*)table, ldt, off,
+                              (__nv_bfloat16*)out, ldo, d));
+    else
+        return mllm_fail(1, "token_side_mid: unknown dtype code %d", dtype);
+    return 0;
+}

@@ -4,12 +4,13 @@
 //   y_c = sum_n S[c, n] C_n + skip_c x_c                          out_c = out_scale * y_c * silu(z_c)
 // x (the convolution's output), B, C and z come in the activation dtype; dt, the decays, the state and the sums are 32-bit.
 //
-// `scan` (prompt portions): a CTA of 128 threads takes 128 / L channels of one request; L lanes share a channel and keep R
-// consecutive state entries each in registers for the whole walk.  Tokens come 16 (8) at a time: the next chunk's inputs
-// are fetched into registers while this one is walked, softplus is taken once per (token, channel) on the way to shared
-// memory, the gate on the way out.  The decays do not depend on the state, so only one fused multiply-add per entry is
-// sequential.  `step` (single tokens): the step size's projection, softplus, update, output and gate in one launch; S, A and
-// the projection's weights are read before the kernel waits for its predecessor.
+// `scan` (prompt portions): a CTA takes 128 / L channels of one request.  128 threads walk: L lanes share a channel and keep R
+// consecutive state entries each in registers throughout; the decays do not depend on the state, so only one fused
+// multiply-add per entry is sequential, and four tokens' sums over the lanes meet together.  128 more threads bring the
+// inputs, three chunks of 16 (8) tokens ahead and through registers, take softplus once per (token, channel) on the way to
+// shared memory, and gate and store the chunk that was walked last: one barrier per chunk.  `step` (single tokens): the step
+// size's projection, softplus, update, output and gate in one launch; S, A and the projection's weights are read before the
+// kernel waits for its predecessor.
 // Every state entry is a recurrence of its own and both kernels do the same operations per token, so the state after some
 // tokens is the same bits however they were cut into portions (single tokens make dt in another summation order).
 #include "common.cuh"
@@ -65,97 +66,159 @@ __device__ __forceinline__ float lanes_sum(float v) {
     return v;
 }
 
-// grid (channel blocks, requests).  x [T][ldx], raw step sizes dt [T][lddt] (32-bit, bias not yet added), bc [T][ldbc] with
-// B at b_off and C at c_off, z [T][ldz], out [T][ldo].
+// grid (channel blocks, requests); the first 128 threads walk the tokens, the other 128 bring and carry away (see the top).
+// x [T][ldx], raw step sizes dt [T][lddt] (32-bit, bias not yet added), bc [T][ldbc] with B at b_off and C at c_off,
+// z [T][ldz], out [T][ldo].
 template <typename T, int L, int R>
-__global__ void __launch_bounds__(THREADS)
+__global__ void __launch_bounds__(2 * THREADS)
 selective_scan_kernel(const T* x, long long ldx, const float* dt, long long lddt, const T* bc, long long ldbc, int b_off,
                       int c_off, const T* z, long long ldz, T* __restrict__ out, long long ldo, SelArgs a) {
-    constexpr int CPB = THREADS / L, NR = L * R, CH = NR > 128 ? 8 : 16;
+    constexpr int CPB = THREADS / L, NR = L * R, CH = (NR > 128 || L == 1) ? 8 : 16;
     constexpr int NB = (CH * NR + THREADS - 1) / THREADS, NX = (CH * CPB + THREADS - 1) / THREADS;
     __shared__ __align__(16) float Bs[2][CH * NR], Cs[2][CH * NR];
-    __shared__ float xs[2][CH * CPB], ds[2][CH * CPB], ys[CH * CPB];
-    const int tid = threadIdx.x, seq = blockIdx.y, base = blockIdx.x * CPB;
+    __shared__ float2 dx[2][CH * CPB];          // (dt, dt * x)
+    __shared__ float ys[2][CH * CPB];
+    const bool walker = threadIdx.x < THREADS;
+    const int tid = threadIdx.x % THREADS, seq = blockIdx.y, base = blockIdx.x * CPB;
     const int ch = tid / L, lane = tid % L, c = base + ch;
-    const bool live = c < a.C;
+    const bool live = walker && c < a.C;
     float ar[R], s[R];
 #pragma unroll
     for (int i = 0; i < R; ++i) {
         const int r = lane * R + i;
         ar[i] = live && r < a.N ? a.A[(size_t)c * a.N + r] * rate_unit<T>() : 0.f;
     }
-    const float skip = live ? a.skip[c] : 0.f;
     pdl_wait();
     pdl_launch();
     const int t0 = a.cu_q[seq], n = a.cu_q[seq + 1] - t0;
     if (n <= 0) return;
+    const int chunks = (n + CH - 1) / CH;
     float* S = a.state + (size_t)a.slots[seq] * a.stride + (size_t)c * a.N;
 #pragma unroll
     for (int i = 0; i < R; ++i) {
         const int r = lane * R + i;
         s[i] = live && r < a.N ? S[r] : 0.f;
     }
-    T rb[NB], rc[NB], rx[NX], rz[NX], rz_next[NX];
-    float rd[NX];
-    auto fetch = [&](int c0) {
-        const int nc = min(CH, n - c0);
+    // what the second half holds between iterations: the raw inputs of the next two chunks to be walked, and z and x of the
+    // two whose results are still to be stored; a load has two iterations to arrive
+    struct In { T b[NB], c[NB], x[NX]; float d[NX]; } in0, in1;
+    struct Out { T z[NX], x[NX]; } out0, out1;
+    const int mine = base + tid % CPB;          // this thread's channel when it brings or carries away
+    const float bias = mine < a.C ? a.bias[mine] : 0.f, skip = mine < a.C ? a.skip[mine] : 0.f;
+    auto fetch = [&](int k, In& r) {
+        if (k >= chunks) return;
+        const int c0 = k * CH, nc = min(CH, n - c0);
 #pragma unroll
         for (int u = 0; u < NB; ++u) {
-            const int i = tid + u * THREADS, tt = i / NR, r = i % NR;
-            const bool ok = i < CH * NR && tt < nc && r < a.N;
+            const int i = tid + u * THREADS, tt = i / NR, e = i % NR;
+            const bool ok = i < CH * NR && tt < nc && e < a.N;
             const T* row = bc + (size_t)(t0 + c0 + (ok ? tt : 0)) * ldbc;
-            rb[u] = ok ? row[b_off + r] : from_f32<T>(0.f);
-            rc[u] = ok ? row[c_off + r] : from_f32<T>(0.f);
+            r.b[u] = ok ? row[b_off + e] : from_f32<T>(0.f);
+            r.c[u] = ok ? row[c_off + e] : from_f32<T>(0.f);
         }
 #pragma unroll
         for (int u = 0; u < NX; ++u) {
-            const int i = tid + u * THREADS, tt = i / CPB, cc = base + i % CPB;
-            const bool ok = i < CH * CPB && tt < nc && cc < a.C;
+            const int i = tid + u * THREADS, tt = i / CPB;
+            const bool ok = i < CH * CPB && tt < nc && mine < a.C;
             const size_t t = t0 + c0 + (ok ? tt : 0);
-            rx[u] = ok ? x[t * ldx + cc] : from_f32<T>(0.f);
-            rz_next[u] = ok ? z[t * ldz + cc] : from_f32<T>(0.f);
-            rd[u] = ok ? dt[t * lddt + cc] + a.bias[cc] : 0.f;
+            r.x[u] = ok ? x[t * ldx + mine] : from_f32<T>(0.f);
+            r.d[u] = ok ? dt[t * lddt + mine] : 0.f;
         }
     };
-    auto put = [&](int buf) {
+    auto put = [&](int k, const In& r) {
+        if (k >= chunks) return;
+        const int buf = k & 1;
 #pragma unroll
         for (int u = 0; u < NB; ++u) {
             const int i = tid + u * THREADS;
-            if (i < CH * NR) { Bs[buf][i] = to_f32(rb[u]); Cs[buf][i] = to_f32(rc[u]); }
+            if (i < CH * NR) { Bs[buf][i] = to_f32(r.b[u]); Cs[buf][i] = to_f32(r.c[u]); }
         }
 #pragma unroll
         for (int u = 0; u < NX; ++u) {
             const int i = tid + u * THREADS;
-            if (i < CH * CPB) { xs[buf][i] = to_f32(rx[u]); ds[buf][i] = softplus_f(rd[u]); }
+            const float d = softplus_f(r.d[u] + bias);
+            if (i < CH * CPB) dx[buf][i] = make_float2(d, d * to_f32(r.x[u]));
         }
     };
-    fetch(0);
-    put(0);
-    for (int c0 = 0, buf = 0; c0 < n; c0 += CH, buf ^= 1) {
-        const int nc = min(CH, n - c0);
-#pragma unroll
-        for (int u = 0; u < NX; ++u) rz[u] = rz_next[u];
-        __syncthreads();                        // this chunk is in; the other buffer and ys are free
-        const bool more = c0 + CH < n;
-        if (more) fetch(c0 + CH);
-        auto walk = [&](int tt) {
-            const float d = ds[buf][tt * CPB + ch], xv = xs[buf][tt * CPB + ch];
-            const float acc = lanes_sum<L>(advance<T, R>(s, ar, d, d * xv, &Bs[buf][tt * NR + lane * R], &Cs[buf][tt * NR + lane * R]));
-            if (lane == 0) ys[tt * CPB + ch] = fmaf(skip, xv, acc);
-        };
-        if (nc == CH) {
-#pragma unroll 4
-            for (int tt = 0; tt < CH; ++tt) walk(tt);
-        } else {
-            for (int tt = 0; tt < nc; ++tt) walk(tt);
-        }
-        if (more) put(buf ^ 1);
-        __syncthreads();
+    auto fetch_out = [&](int k, Out& o) {
+        if (k >= chunks) return;
+        const int c0 = k * CH, nc = min(CH, n - c0);
 #pragma unroll
         for (int u = 0; u < NX; ++u) {
-            const int i = tid + u * THREADS, tt = i / CPB, cc = base + i % CPB;
-            if (i < CH * CPB && tt < nc && cc < a.C)
-                out[(size_t)(t0 + c0 + tt) * ldo + cc] = from_f32<T>(ys[i] * silu_f(to_f32(rz[u])) * a.out_scale);
+            const int i = tid + u * THREADS, tt = i / CPB;
+            const bool ok = i < CH * CPB && tt < nc && mine < a.C;
+            const size_t t = t0 + c0 + (ok ? tt : 0);
+            o.z[u] = ok ? z[t * ldz + mine] : from_f32<T>(0.f);
+            o.x[u] = ok ? x[t * ldx + mine] : from_f32<T>(0.f);
+        }
+    };
+    auto put_out = [&](int k, const Out& o) {
+        if (k < 0) return;
+        const int c0 = k * CH, nc = min(CH, n - c0);
+#pragma unroll
+        for (int u = 0; u < NX; ++u) {
+            const int i = tid + u * THREADS, tt = i / CPB;
+            if (i < CH * CPB && tt < nc && mine < a.C)
+                out[(size_t)(t0 + c0 + tt) * ldo + mine] =
+                    from_f32<T>(fmaf(skip, to_f32(o.x[u]), ys[k & 1][i]) * silu_f(to_f32(o.z[u])) * a.out_scale);
+        }
+    };
+    auto bring = [&](int k, In& next, Out& done) {          // next: chunk k + 1; done: chunk k - 1
+        put(k + 1, next);
+        put_out(k - 1, done);
+        fetch(k + 3, next);
+        fetch_out(k + 1, done);
+    };
+    auto walk = [&](int k) {
+        const int nc = min(CH, n - k * CH);
+        const float2* dk = dx[k & 1] + ch;
+        const float *bk = Bs[k & 1] + lane * R, *ck = Cs[k & 1] + lane * R;
+        float* yk = ys[k & 1] + ch;
+        auto token = [&](int tt) {
+            const float2 d = dk[tt * CPB];
+            return advance<T, R>(s, ar, d.x, d.y, bk + tt * NR, ck + tt * NR);
+        };
+        if (L >= 4 && nc == CH) {
+            // four tokens together: their sums over the L lanes meet by halving, and a lane ends with one token's.  Nothing is
+            // stored before the whole chunk has been walked, so that later tokens' loads are not held up.
+            const bool up1 = lane & (L / 2), up2 = lane & (L / 4);
+            float w[CH / 4];
+#pragma unroll
+            for (int q = 0; q < CH / 4; ++q) {
+                const float v0 = token(4 * q), v1 = token(4 * q + 1), v2 = token(4 * q + 2), v3 = token(4 * q + 3);
+                const float h0 = (up1 ? v2 : v0) + __shfl_xor_sync(0xffffffffu, up1 ? v0 : v2, L / 2);
+                const float h1 = (up1 ? v3 : v1) + __shfl_xor_sync(0xffffffffu, up1 ? v1 : v3, L / 2);
+                w[q] = (up2 ? h1 : h0) + __shfl_xor_sync(0xffffffffu, up2 ? h0 : h1, L / 4);
+#pragma unroll
+                for (int o = L / 8; o > 0; o >>= 1) w[q] += __shfl_xor_sync(0xffffffffu, w[q], o);
+            }
+            if (L == 4 || (lane & (L / 4 - 1)) == 0) {
+                const int at = (up1 ? 2 : 0) + (up2 ? 1 : 0);
+#pragma unroll
+                for (int q = 0; q < CH / 4; ++q) yk[(4 * q + at) * CPB] = w[q];
+            }
+            return;
+        }
+        for (int tt = 0; tt < nc; ++tt) {
+            const float w = lanes_sum<L>(token(tt));
+            if (lane == 0) yk[tt * CPB] = w;
+        }
+    };
+    if (!walker) {
+        fetch(0, in0);
+        fetch(1, in1);
+        put(0, in0);
+        fetch(2, in0);
+        fetch_out(0, out0);
+    }
+    for (int k = 0; k <= chunks; ++k) {
+        __syncthreads();                        // chunk k is in; what was walked last is complete
+        if (walker) {
+            if (k < chunks) walk(k);
+        } else if (k & 1) {                     // chunk k + 1 came into in0, chunk k - 1's outputs wait for out0
+            bring(k, in0, out0);
+        } else {
+            bring(k, in1, out1);
         }
     }
     if (a.write_state && live) {
@@ -251,7 +314,7 @@ template <typename T>
 int scan_launch(const void* x, long long ldx, const float* dt, long long lddt, const void* bc, long long ldbc, int b_off, int c_off,
                 const void* z, long long ldz, void* out, long long ldo, int S, const SelArgs& a, cudaStream_t stream) {
 #define MLLM_GO(L, R)                                                                                                    \
-    MLLM_CUDA(mllm_launch(selective_scan_kernel<T, L, R>, dim3((a.C + THREADS / L - 1) / (THREADS / L), S), dim3(THREADS), 0, \
+    MLLM_CUDA(mllm_launch(selective_scan_kernel<T, L, R>, dim3((a.C + THREADS / L - 1) / (THREADS / L), S), dim3(2 * THREADS), 0, \
                           stream, true, (const T*)x, ldx, dt, lddt, (const T*)bc, ldbc, b_off, c_off, (const T*)z, ldz,  \
                           (T*)out, ldo, a))
     MLLM_BY_LANES(MLLM_GO);

@@ -31,7 +31,7 @@ template <typename T, typename TO>
 __global__ void __launch_bounds__(256)
 conv_silu_kernel(const T* proj, long long ld, int off, const float* __restrict__ w, const float* __restrict__ bias,
                  const float* state, long long state_stride, int conv_off, const int* token_seq, const int* cu_q,
-                 const int* slots, TO* out, int Tn, int C, int taps) {
+                 const int* slots, TO* out, long long ldo, int Tn, int C, int taps) {
     pdl_wait();
     const int t = blockIdx.y, ch = blockIdx.x * 256 + threadIdx.x;
     if (ch >= C) return;
@@ -50,7 +50,7 @@ conv_silu_kernel(const T* proj, long long ld, int off, const float* __restrict__
             acc = fmaf(w[(size_t)ch * taps + j], u, acc);
         }
     }
-    out[(size_t)t * C + ch] = from_f32<TO>(silu_f(acc));
+    out[(size_t)t * ldo + ch] = from_f32<TO>(silu_f(acc));
 }
 
 // Steps in which every request brings one token: grid (channel blocks, requests); a thread computes its channel's output
@@ -58,8 +58,8 @@ conv_silu_kernel(const T* proj, long long ld, int off, const float* __restrict__
 template <typename T, typename TO>
 __global__ void __launch_bounds__(256)
 conv_step_kernel(const T* proj, long long ld, int off, const float* __restrict__ w, const float* __restrict__ bias,
-                 float* state, long long state_stride, int conv_off, const int* cu_q, const int* slots, TO* out, int C,
-                 int taps, int write_state) {
+                 float* state, long long state_stride, int conv_off, const int* cu_q, const int* slots, TO* out,
+                 long long ldo, int C, int taps, int write_state) {
     pdl_wait();
     const int ch = blockIdx.x * 256 + threadIdx.x, s = blockIdx.y;
     if (ch >= C) return;
@@ -76,7 +76,7 @@ conv_step_kernel(const T* proj, long long ld, int off, const float* __restrict__
         }
     }
     acc = fmaf(w[(size_t)ch * taps + taps - 1], u, acc);
-    out[(size_t)t * C + ch] = from_f32<TO>(silu_f(acc));
+    out[(size_t)t * ldo + ch] = from_f32<TO>(silu_f(acc));
     if (write_state) {
 #pragma unroll
         for (int k = 0; k < MAX_TAPS; ++k) {
@@ -277,22 +277,22 @@ int scan_launch(int rows, dim3 grid, size_t smem, cudaStream_t stream, const flo
 MLLM_EXPORT int mllm_ssd_max_state_rows() { return 256; }
 MLLM_EXPORT int mllm_ssd_max_taps() { return MAX_TAPS; }
 
-// The convolution of the step's tokens (out [T][C] 32-bit, or in `dtype` when out_act is 1), then the update of the requests'
+// The convolution of the step's tokens (out [T][ldo] 32-bit, or in `dtype` when out_act is 1), then the update of the requests'
 // conv states.
 namespace {
 template <typename T, typename TO>
 int conv_launch(const void* proj, long long ld, int off, const float* w, const float* bias, float* state, long long state_stride,
-                int conv_off, const int* token_seq, const int* cu_q, const int* slots, void* out, int Tn, int S, int C, int taps,
-                int write_state, cudaStream_t stream) {
+                int conv_off, const int* token_seq, const int* cu_q, const int* slots, void* out, long long ldo, int Tn, int S, int C,
+                int taps, int write_state, cudaStream_t stream) {
     const dim3 grid((C + 255) / 256, Tn);
     const dim3 ugrid((C + 255) / 256, S);
     if (Tn == S) {                          // one token per request: output and state update in one launch
         MLLM_CUDA(mllm_launch(conv_step_kernel<T, TO>, ugrid, dim3(256), 0, stream, true, (const T*)proj, ld, off, w, bias, state,
-                              state_stride, conv_off, cu_q, slots, (TO*)out, C, taps, write_state));
+                              state_stride, conv_off, cu_q, slots, (TO*)out, ldo, C, taps, write_state));
         return 0;
     }
     MLLM_CUDA(mllm_launch(conv_silu_kernel<T, TO>, grid, dim3(256), 0, stream, true, (const T*)proj, ld, off, w, bias,
-                          (const float*)state, state_stride, conv_off, token_seq, cu_q, slots, (TO*)out, Tn, C, taps));
+                          (const float*)state, state_stride, conv_off, token_seq, cu_q, slots, (TO*)out, ldo, Tn, C, taps));
     if (write_state && taps > 1)
         MLLM_CUDA(mllm_launch(conv_state_update_kernel<T>, ugrid, dim3(256), 0, stream, true, (const T*)proj, ld, off, state,
                               state_stride, conv_off, cu_q, slots, C, taps));
@@ -302,20 +302,20 @@ int conv_launch(const void* proj, long long ld, int off, const float* w, const f
 
 MLLM_EXPORT int mllm_ssd_conv(const void* proj, long long ld, int off, const float* w, const float* bias, float* state,
                               long long state_stride, int conv_off, const int* token_seq, const int* cu_q, const int* slots,
-                              void* out, int out_act, int Tn, int S, int C, int taps, int write_state, int dtype,
+                              void* out, long long ldo, int out_act, int Tn, int S, int C, int taps, int write_state, int dtype,
                               cudaStream_t stream) {
     if (Tn <= 0 || C <= 0) return 0;
     if (taps < 1 || taps > MAX_TAPS) return mllm_fail(1, "ssd_conv: %d taps (1 to %d)", taps, MAX_TAPS);
     if (Tn > 65535 || S > 65535) return mllm_fail(1, "ssd_conv: more than 65535 tokens in a step");
     using bf = __nv_bfloat16;
     if (dtype == MLLM_F32)
-        return conv_launch<float, float>(proj, ld, off, w, bias, state, state_stride, conv_off, token_seq, cu_q, slots, out, Tn, S, C,
+        return conv_launch<float, float>(proj, ld, off, w, bias, state, state_stride, conv_off, token_seq, cu_q, slots, out, ldo, Tn, S, C,
                                          taps, write_state, stream);
     if (dtype == MLLM_BF16 && out_act)
-        return conv_launch<bf, bf>(proj, ld, off, w, bias, state, state_stride, conv_off, token_seq, cu_q, slots, out, Tn, S, C, taps,
+        return conv_launch<bf, bf>(proj, ld, off, w, bias, state, state_stride, conv_off, token_seq, cu_q, slots, out, ldo, Tn, S, C, taps,
                                    write_state, stream);
     if (dtype == MLLM_BF16)
-        return conv_launch<bf, float>(proj, ld, off, w, bias, state, state_stride, conv_off, token_seq, cu_q, slots, out, Tn, S, C,
+        return conv_launch<bf, float>(proj, ld, off, w, bias, state, state_stride, conv_off, token_seq, cu_q, slots, out, ldo, Tn, S, C,
                                       taps, write_state, stream);
     return mllm_fail(1, "ssd_conv: unknown dtype code %d", dtype);
 }

@@ -42,6 +42,8 @@ def _signatures(lib):
     lib.mllm_set_pdl.restype = c_int
     sig = {
         "mllm_token_side_gate": [c_void_p, c_ll, c_void_p, c_void_p, c_ll, c_int, c_void_p, c_ll, c_int, c_int, c_int, c_void_p],
+        "mllm_token_side_mid": [c_void_p, c_ll, c_void_p, c_int, c_void_p, c_void_p, c_ll, c_int, c_void_p, c_ll, c_int, c_int, c_int,
+                                c_void_p],
         "mllm_embed": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p],
         "mllm_concat_terms": [c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_ll, c_int, c_int, c_int, c_int, c_void_p],
         "mllm_resolve_tokens": [c_void_p, c_int, c_void_p, c_int, c_void_p],
@@ -139,7 +141,7 @@ def _signatures(lib):
                                       c_int, c_int, c_int, c_float, c_void_p, c_void_p],
         "mllm_latent_mma_ok": [c_int, c_int, c_int],
         "mllm_ssd_conv": [c_void_p, c_ll, c_int, c_void_p, c_void_p, c_void_p, c_ll, c_int, c_void_p, c_void_p, c_void_p,
-                          c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+                          c_void_p, c_ll, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
         "mllm_ssd_scan": [c_void_p, c_int, c_int, c_int, c_void_p, c_ll, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_ll,
                           c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
         "mllm_gated_group_norm": [c_void_p, c_void_p, c_ll, c_void_p, c_void_p, c_ll, c_int, c_int, c_int, c_float, c_int,
@@ -413,6 +415,25 @@ def token_side_gate(z, ids, table, off: int, out) -> None:
         raise KernelError(f"token_side_gate: z {tuple(z.shape)}, table {tuple(table.shape)} from column {off}, out {tuple(out.shape)}")
     _call("mllm_token_side_gate", z.data_ptr(), _rows("z", z), ids.data_ptr(), table.data_ptr(), table.shape[1], int(off),
           out.data_ptr(), _rows("out", out), T, d, _dt(table), _stream())
+
+
+SIDE_FEW_TOKENS, SIDE_MAX_WIDTH = 16, 12288      # what csrc/embedding.cu's single-launch kernel is for
+
+
+def token_side_mid(h, weight, ids, table, off: int, out) -> None:
+    """out[t, c] = gelu_tanh(weight[c] . h[t]) * table[ids[t], off + c] in one launch, for few tokens: h [T, D] (at most
+    ``SIDE_MAX_WIDTH`` wide), weight [d, D], table and out [T, d] in one dtype."""
+    _cuda("h", h, contiguous=False)
+    _cuda("weight", weight, h.dtype)
+    _cuda("ids", ids, torch.int32)
+    _cuda("table", table, h.dtype)
+    _cuda("out", out, h.dtype, contiguous=False)
+    T, D = h.shape
+    d = weight.shape[0]
+    if weight.shape[1] != D or ids.numel() != T or tuple(out.shape) != (T, d) or off < 0 or off + d > table.shape[1] or D > SIDE_MAX_WIDTH:
+        raise KernelError(f"token_side_mid: h {tuple(h.shape)}, weight {tuple(weight.shape)}, table {tuple(table.shape)} from column {off}")
+    _call("mllm_token_side_mid", h.data_ptr(), _rows("h", h), weight.data_ptr(), D, ids.data_ptr(), table.data_ptr(), table.shape[1],
+          int(off), out.data_ptr(), _rows("out", out), T, d, _dt(h), _stream())
 
 
 def concat_terms(x, x0, out, terms: int) -> None:
@@ -1733,7 +1754,7 @@ def ssd_conv(proj, off: int, weight, bias, state, conv_off: int, ctx, out, *, wr
     _cuda("weight", weight, torch.float32)
     _cuda("bias", bias, torch.float32)
     _cuda("state", state, torch.float32)
-    _cuda("out", out)
+    _cuda("out", out, contiguous=False)
     if out.dtype not in (torch.float32, proj.dtype):
         raise KernelError(f"ssd_conv: out {out.dtype} for {proj.dtype} inputs")
     C, taps = weight.shape
@@ -1742,7 +1763,7 @@ def ssd_conv(proj, off: int, weight, bias, state, conv_off: int, ctx, out, *, wr
         raise KernelError("ssd_conv: shapes do not fit")
     _call("mllm_ssd_conv", proj.data_ptr(), _rows("proj", proj), int(off), weight.data_ptr(), bias.data_ptr(), state.data_ptr(),
           state.stride(0), int(conv_off), ctx.token_seq.data_ptr(), ctx.cu_q.data_ptr(), ctx.state_slots.data_ptr(),
-          out.data_ptr(), int(out.dtype == proj.dtype), T, ctx.S, C, taps, int(write_state), _dt(proj), _stream())
+          out.data_ptr(), _rows("out", out), int(out.dtype == proj.dtype), T, ctx.S, C, taps, int(write_state), _dt(proj), _stream())
     if write_state and taps > 1 and T != ctx.S:
         global launches
         launches += 1       # the state's update (steps of single tokens do both in one launch)

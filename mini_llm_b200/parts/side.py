@@ -40,10 +40,13 @@ class TokenSideBranch(TokenSide):
         import torch
         ops = self.rt.ops
         T = h.shape[0]
-        z = ctx.ws.buf("side_gate", T, -(-self.dim // 8) * 8, torch.float32)[:, :self.dim]
-        ops.linear(h, self.gate_weight, None, out=z)
         mid = ctx.ws.buf("side_mid", T, -(-self.dim // 8) * 8, self.rt.act_dtype)[:, :self.dim]    # rows stay 16-byte aligned
-        ops.token_side_gate(z, ctx.token_ids, self.source.table, self.part * self.dim, mid)
+        if T <= ops.SIDE_FEW_TOKENS and self.hidden_size <= ops.SIDE_MAX_WIDTH:      # few tokens: one launch
+            ops.token_side_mid(h, self.gate_weight, ctx.token_ids, self.source.table, self.part * self.dim, mid)
+        else:
+            z = ctx.ws.buf("side_gate", T, -(-self.dim // 8) * 8, torch.float32)[:, :self.dim]
+            ops.linear(h, self.gate_weight, None, out=z)
+            ops.token_side_gate(z, ctx.token_ids, self.source.table, self.part * self.dim, mid)
         ops.linear(mid, self.proj_weight, None, out=y)
 
 
