@@ -35,6 +35,12 @@ struct SelArgs {
 __device__ __forceinline__ float softplus_f(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
 __device__ __forceinline__ float silu_f(float v) { return v / (1.0f + expf(-v)); }
 
+// silu for a result that is rounded to T: with bfloat16 the fast exponential and division (about 1e-6) are far below that rounding
+template <typename T> __device__ __forceinline__ float silu_out(float v) {
+    if constexpr (sizeof(T) == 4) return silu_f(v);
+    return __fdividef(v, 1.0f + __expf(-v));
+}
+
 // exp(dt * a): on the bfloat16 path the rates are kept in units of ln 2 and the exponential is one instruction
 template <typename T> __device__ __forceinline__ float rate_unit() { return sizeof(T) == 4 ? 1.0f : LOG2E; }
 template <typename T> __device__ __forceinline__ float decay_of(float dt, float a) {
@@ -105,24 +111,30 @@ selective_scan_kernel(const T* x, long long ldx, const float* dt, long long lddt
     struct Out { T z[NX], x[NX]; } out0, out1;
     const int mine = base + tid % CPB;          // this thread's channel when it brings or carries away
     const float bias = mine < a.C ? a.bias[mine] : 0.f, skip = mine < a.C ? a.skip[mine] : 0.f;
+    // Row numbers and columns are held inside the tensors instead of asking before every load: what a token beyond the portion
+    // or a channel beyond the last brings is never used.  Token tid / CPB + u * L of a chunk, one channel throughout.
+    const int mine_in = min(mine, a.C - 1), first = tid / CPB;
+    const char* px = reinterpret_cast<const char*>(x + (size_t)t0 * ldx + mine_in);
+    const char* pz = reinterpret_cast<const char*>(z + (size_t)t0 * ldz + mine_in);
+    const char* pd = reinterpret_cast<const char*>(dt + (size_t)t0 * lddt + mine_in);
+    const char* pb = reinterpret_cast<const char*>(bc + (size_t)t0 * ldbc + b_off);
+    const ptrdiff_t to_c = (ptrdiff_t)(c_off - b_off) * (ptrdiff_t)sizeof(T);
+    const unsigned sx = (unsigned)(ldx * sizeof(T)), sz = (unsigned)(ldz * sizeof(T)), sd = (unsigned)(lddt * 4), sb = (unsigned)(ldbc * sizeof(T));
+    auto at = [](const char* p, unsigned row, unsigned stride) { return p + (unsigned long long)row * stride; };
     auto fetch = [&](int k, In& r) {
         if (k >= chunks) return;
-        const int c0 = k * CH, nc = min(CH, n - c0);
 #pragma unroll
         for (int u = 0; u < NB; ++u) {
-            const int i = tid + u * THREADS, tt = i / NR, e = i % NR;
-            const bool ok = i < CH * NR && tt < nc && e < a.N;
-            const T* row = bc + (size_t)(t0 + c0 + (ok ? tt : 0)) * ldbc;
-            r.b[u] = ok ? row[b_off + e] : from_f32<T>(0.f);
-            r.c[u] = ok ? row[c_off + e] : from_f32<T>(0.f);
+            const int i = tid + u * THREADS, e = i % NR;
+            const char* row = at(pb, min(k * CH + i / NR, n - 1), sb) + min(e, a.N - 1) * (int)sizeof(T);
+            r.b[u] = *reinterpret_cast<const T*>(row);
+            r.c[u] = *reinterpret_cast<const T*>(row + to_c);
         }
 #pragma unroll
         for (int u = 0; u < NX; ++u) {
-            const int i = tid + u * THREADS, tt = i / CPB;
-            const bool ok = i < CH * CPB && tt < nc && mine < a.C;
-            const size_t t = t0 + c0 + (ok ? tt : 0);
-            r.x[u] = ok ? x[t * ldx + mine] : from_f32<T>(0.f);
-            r.d[u] = ok ? dt[t * lddt + mine] : 0.f;
+            const unsigned t = min(k * CH + first + u * L, n - 1);
+            r.x[u] = *reinterpret_cast<const T*>(at(px, t, sx));
+            r.d[u] = *reinterpret_cast<const float*>(at(pd, t, sd));
         }
     };
     auto put = [&](int k, const In& r) {
@@ -131,7 +143,8 @@ selective_scan_kernel(const T* x, long long ldx, const float* dt, long long lddt
 #pragma unroll
         for (int u = 0; u < NB; ++u) {
             const int i = tid + u * THREADS;
-            if (i < CH * NR) { Bs[buf][i] = to_f32(r.b[u]); Cs[buf][i] = to_f32(r.c[u]); }
+            const bool ok = i % NR < a.N;               // entries beyond the state stay zero
+            if (i < CH * NR) { Bs[buf][i] = ok ? to_f32(r.b[u]) : 0.f; Cs[buf][i] = ok ? to_f32(r.c[u]) : 0.f; }
         }
 #pragma unroll
         for (int u = 0; u < NX; ++u) {
@@ -142,25 +155,23 @@ selective_scan_kernel(const T* x, long long ldx, const float* dt, long long lddt
     };
     auto fetch_out = [&](int k, Out& o) {
         if (k >= chunks) return;
-        const int c0 = k * CH, nc = min(CH, n - c0);
 #pragma unroll
         for (int u = 0; u < NX; ++u) {
-            const int i = tid + u * THREADS, tt = i / CPB;
-            const bool ok = i < CH * CPB && tt < nc && mine < a.C;
-            const size_t t = t0 + c0 + (ok ? tt : 0);
-            o.z[u] = ok ? z[t * ldz + mine] : from_f32<T>(0.f);
-            o.x[u] = ok ? x[t * ldx + mine] : from_f32<T>(0.f);
+            const unsigned t = min(k * CH + first + u * L, n - 1);
+            o.z[u] = *reinterpret_cast<const T*>(at(pz, t, sz));
+            o.x[u] = *reinterpret_cast<const T*>(at(px, t, sx));
         }
     };
+    char* po = reinterpret_cast<char*>(out + (size_t)t0 * ldo + mine_in);
+    const unsigned so = (unsigned)(ldo * sizeof(T));
     auto put_out = [&](int k, const Out& o) {
-        if (k < 0) return;
-        const int c0 = k * CH, nc = min(CH, n - c0);
+        if (k < 0 || mine >= a.C) return;
 #pragma unroll
         for (int u = 0; u < NX; ++u) {
-            const int i = tid + u * THREADS, tt = i / CPB;
-            if (i < CH * CPB && tt < nc && mine < a.C)
-                out[(size_t)(t0 + c0 + tt) * ldo + mine] =
-                    from_f32<T>(fmaf(skip, to_f32(o.x[u]), ys[k & 1][i]) * silu_f(to_f32(o.z[u])) * a.out_scale);
+            const int i = tid + u * THREADS, t = k * CH + first + u * L;
+            if (i < CH * CPB && t < n)
+                *reinterpret_cast<T*>(po + (unsigned long long)(unsigned)t * so) =
+                    from_f32<T>(fmaf(skip, to_f32(o.x[u]), ys[k & 1][i]) * silu_out<T>(to_f32(o.z[u])) * a.out_scale);
         }
     };
     auto bring = [&](int k, In& next, Out& done) {          // next: chunk k + 1; done: chunk k - 1
@@ -276,7 +287,7 @@ selective_step_kernel(const T* x, long long ldx, const T* low, long long ldlow, 
     const float d = softplus_f(lanes_sum<L>(acc) + bias);
     const float y = lanes_sum<L>(advance<T, R>(s, ar, d, d * xv, Bs + lane * R, Cs + lane * R));
     if (!live) return;
-    if (lane == 0) out[(size_t)t * ldo + c] = from_f32<T>(fmaf(skip, xv, y) * silu_f(zv) * a.out_scale);
+    if (lane == 0) out[(size_t)t * ldo + c] = from_f32<T>(fmaf(skip, xv, y) * silu_out<T>(zv) * a.out_scale);
     if (a.write_state) {
 #pragma unroll
         for (int i = 0; i < R; ++i)
@@ -286,6 +297,7 @@ selective_step_kernel(const T* x, long long ldx, const T* low, long long ldlow, 
 
 int check(const char* what, const SelArgs& a, int S) {
     if (a.C <= 0 || a.N <= 0 || a.N > 256) return mllm_fail(1, "%s: %d channels with states of %d entries (at most 256)", what, a.C, a.N);
+    if (a.C > (1 << 26)) return mllm_fail(1, "%s: %d channels", what, a.C);
     if (a.stride < (long long)a.C * a.N) return mllm_fail(1, "%s: state rows of %lld floats", what, a.stride);
     if (S > 65535) return mllm_fail(1, "%s: more than 65535 requests in a step", what);
     return 0;
@@ -348,6 +360,8 @@ MLLM_EXPORT int mllm_selective_scan(const void* x, long long ldx, const float* d
     if (S <= 0) return 0;
     SelArgs a{A, skip, bias, state, stride, cu_q, slots, C, N, write_state, out_scale};
     if (int rc = check("selective_scan", a, S)) return rc;
+    for (long long ld : {ldx, lddt, ldbc, ldz, ldo})
+        if (ld <= 0 || ld >= (1ll << 30)) return mllm_fail(1, "selective_scan: rows of %lld entries", ld);
     if (dtype == MLLM_F32) return scan_launch<float>(x, ldx, dt, lddt, bc, ldbc, b_off, c_off, z, ldz, out, ldo, S, a, stream);
     if (dtype == MLLM_BF16) return scan_launch<__nv_bfloat16>(x, ldx, dt, lddt, bc, ldbc, b_off, c_off, z, ldz, out, ldo, S, a, stream);
     return mllm_fail(1, "selective_scan: unknown dtype code %d", dtype);
