@@ -1,6 +1,6 @@
-// Retention: linear attention with a fixed decay per head.  With q_t, k_t rows of dk entries (rotated) and v_t of dv:
-//   S_t = decay_h S_(t-1) + k_t v_t^T          o_t = S_t^T q_t          S [dk, dv], zero at the start of a sequence
-//   y_t = o_t / sqrt(mean(o_t^2) + eps) * silu(g_t)                      per head, no weight
+// Retention (RetNet): a matrix memory S [dk, dv] per head that forgets at a constant rate a_h.  With turned rows q, k of dk
+// entries, v of dv and a gate row g, token after token from S = 0:
+//   S <- a_h S + k v^T          o = S^T q          y = o / sqrt(mean(o^2) + eps) * silu(g)
 // The projections come in 32-bit; everything here is 32-bit.  A request's state is S of every head in one row.
 //
 // `rotate_heads` turns the first rot_dims entries of every query and key head by position * freq[i] in place (entry i pairs

@@ -1,7 +1,7 @@
-// The selective scan with a state per channel (Mamba's first form).  Per channel c and state entry n, S zero at the start:
-//   dt_c = softplus(raw_c + bias_c)
-//   S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n          A negative: [C, N] rates
-//   y_c = sum_n S[c, n] C_n + skip_c x_c                          out_c = out_scale * y_c * silu(z_c)
+// The selective scan with a state vector per channel (Mamba's first form).  A channel with rates a in R^N (negative), a skip
+// factor d and a state s in R^N (at first zeros) takes, token after token, an input x, a gate z, a raw step size and the two
+// vectors B, C that all channels of the token share:
+//   h = softplus(raw + bias)        s <- e^(h a) * s + h x B   (entry by entry)        out = out_scale * (s . C + d x) * silu(z)
 // x (the convolution's output), B, C and z come in the activation dtype; dt, the decays, the state and the sums are 32-bit.
 //
 // `scan` (prompt portions): a CTA takes 128 / L channels of one request.  128 threads walk: L lanes share a channel and keep R
@@ -21,7 +21,7 @@ constexpr int THREADS = 128;
 constexpr float LOG2E = 1.4426950408889634f;
 
 struct SelArgs {
-    const float* A;                 // [C][N]
+    const float* A;                 // [C][N] the channels' rates
     const float* skip;              // [C]
     const float* bias;              // [C] of the step sizes
     float* state;                   // [slots][stride]: S [C][N] at the row's start

@@ -1651,7 +1651,7 @@ def rotate_heads(proj, q_off: int, k_off: int, ctx, *, heads: int, dim: int, fre
 
 def retention_scan(proj, cols: dict, decay, state, ctx, raw, *, heads: int, dim: int, vdim: int, write_state: bool = True,
                    want_cols: int = 0) -> None:
-    """S <- decay_h S + k v^T, raw = S^T q over the step's tokens, request by request and head by head.  proj 32-bit [T, .] with
+    """S <- a_h S + k v^T (a_h: ``decay``), raw = S^T q over the step's tokens, request by request and head by head.  proj 32-bit [T, .] with
     the columns ``cols`` = {"q", "k", "v"} -> first column (queries and keys already rotated); decay float32 [heads]; state
     [slots, >= heads * dim * vdim]: S [heads, dim, vdim]; raw [T, heads * vdim] 32-bit."""
     _retention_sizes("retention_scan", proj, {c: cols[c] for c in "qkv"}, decay, state, heads, dim, vdim)
@@ -1714,10 +1714,10 @@ def _selective_sizes(name: str, x, bc, b_off, c_off, z, A, skip, dt_bias, state,
 
 def selective_scan(x, dt, bc, b_off: int, c_off: int, z, A, skip, dt_bias, state, ctx, out, *, out_scale: float = 1.0,
                    write_state: bool = True) -> None:
-    """The selective scan with a state per channel over the step's tokens, request by request: d = softplus(dt + dt_bias);
-    S[c, n] <- exp(d_c A[c, n]) S[c, n] + d_c x_c B_n; out_c = out_scale * (sum_n S[c, n] C_n + skip_c x_c) * silu(z_c).
+    """The selective scan with a state vector s per channel over the step's tokens, request by request: h = softplus(dt +
+    dt_bias); s <- exp(h a) * s + h x B with a the channel's row of A; out = out_scale * (s . C + skip x) * silu(z).
     x, z, out [T, C] and bc [T, .] (B at column b_off, C at c_off) in one dtype; dt float32 [T, C]; A float32 [C, N] (negative);
-    state [slots, >= C * N]: S [C, N]."""
+    state [slots, >= C * N]: the channels' s one after the other."""
     T, C, N = _selective_sizes("selective_scan", x, bc, b_off, c_off, z, A, skip, dt_bias, state, out)
     _cuda("dt", dt, torch.float32, contiguous=False)
     if tuple(dt.shape) != (T, C):

@@ -1,13 +1,13 @@
-"""Retention: linear attention with a fixed decay per head, without softmax or denominator.
+"""Retention (RetNet): a matrix memory per head that forgets at a constant rate.
 
-q = W_q h, k = W_k h (heads of ``head_dim``), v = W_v h (heads of ``v_head_dim``), no biases; queries and keys turn by their
-position (``rot_dims`` entries of every head, ``parts.rotary``) and the keys are multiplied by head_dim^(-1/2) afterwards.
-Per head, with a state S [dim, vdim] that starts at zero and the head's constant decay a:
+Queries and keys (heads of ``head_dim`` entries, bias-free projections) are turned by their position (``rot_dims`` entries,
+``parts.rotary``) and the turned keys scaled by head_dim^(-1/2); values are heads of ``v_head_dim``.  A head with the constant
+a keeps S [dim, vdim], at first all zeros:
 
-    S_t = a S_(t-1) + k_t v_t^T        o_t = S_t^T q_t
+    S <- a S + k v^T        o = S^T q
 
-Each head's o_t is divided by its root mean square (eps inside the root, no weight); the joined heads are multiplied by
-silu(W_g h), then W_o.  The four input matrices are one product whose result stays 32-bit (its columns enter the recurrence);
+o is brought to unit root mean square (eps inside the root) head by head, gated with silu of a fourth projection, and
+projected by W_o.  The four input matrices are one product whose result stays 32-bit (its columns enter the recurrence);
 the rotation, the state, o, the norm and the gate are 32-bit whatever the engine's dtype.  The request's state is S of every
 head in one row of the cache manager's state arena.
 """

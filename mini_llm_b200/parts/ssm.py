@@ -80,13 +80,15 @@ register_part("mixer", "mamba2", Mamba2Mixer)
 
 
 class MambaMixer(ProjectedMixer):
-    """The selective scan with a state per channel (Mamba's first form).  W_in h is [x: inner | z: inner]; x passes the causal
-    convolution per channel (weights [inner, taps], a bias) and silu; W_x x is [dt: rank | B: N | C: N];
-    dt <- softplus(W_dt dt + bias), one per channel; A = -exp(A_log) [inner, N].  Per channel c, S zero at the start:
+    """The selective scan with a state vector per channel (Mamba's first form).  One product gives ``inner`` inputs and as many
+    gates z; the inputs go through Mamba-2's short convolution (with bias and silu) to x; a second product of x gives, side by
+    side, a low-rank step size of ``dt_rank`` numbers and the vectors B and C of ``state_size`` entries; a third one spreads the
+    step size over the channels, h = softplus(W_dt low + bias).  Channel c with the rates a = -exp(A_log[c]) keeps s, at first
+    zeros:
 
-        S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n        y_c = sum_n S[c, n] C_n + D_c x_c
+        s <- e^(h a) * s + h x B   (entry by entry)        y = s . C + D_c x
 
-    and W_o (y * silu(z)).  The request's state holds S and the last taps - 1 inputs of the convolution, both 32-bit, in one
+    and the mixer's result is W_o (y * silu(z)).  The request's state holds the channels' s and the last taps - 1 inputs of the convolution, both 32-bit, in one
     row of the cache manager's state arena; dt, the decays, the recurrence and the gate are 32-bit whatever the engine's
     dtype."""
 

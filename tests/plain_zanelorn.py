@@ -55,9 +55,9 @@ def softplus(z):
 
 # ------------------------------------------------------------------------------------------- rotation
 def rotate_halves(x, positions, dims: int, base: float, factor: float = 1.0):
-    """x [..., T, d]: entry i and entry i + dims/2 of the first ``dims`` are a pair (u, v); at position p it becomes
-    (u cos a - v sin a, v cos a + u sin a), a = p * base^(-2i/dims) / factor.  The angle is taken in 32-bit: frequency and
-    position as float32, their product rounded to float32."""
+    """x [..., T, d]: entries i and i + dims/2 of the first ``dims``, read as one complex number, are multiplied by e^(j a),
+    a = position * base^(-2i/dims) / factor.  The angle is taken in 32-bit: frequency and position as float32, their product
+    rounded to float32."""
     if dims == 0:
         return x
     half = dims // 2
@@ -70,7 +70,7 @@ def rotate_halves(x, positions, dims: int, base: float, factor: float = 1.0):
 
 # ------------------------------------------------------------------------------------------- retention
 def retention_scan(q, k, v, decay: Sequence[float], state=None):
-    """Per head, S zero at the start: S <- decay_h S + k v^T, o = S^T q.  q, k [T, Hr, dk], v [T, Hr, dv]; returns
+    """Head by head, from S = 0: S <- a_h S + k v^T (a_h: ``decay``), o = S^T q.  q, k [T, Hr, dk], v [T, Hr, dv]; returns
     (o [T, Hr, dv], S)."""
     T, Hr, dk = q.shape
     dv = v.shape[2]
@@ -144,7 +144,7 @@ def causal_conv(x, weight, bias):
 
 
 def selective_scan(x, dt, A, B, C, skip, state=None):
-    """S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n; y_c = sum_n S[c, n] C_n + skip_c x_c.  x, dt [T, channels],
+    """Every channel's row s of S: s <- e^(dt a) * s + dt x B (a its row of A), y = s . C + skip x.  x, dt [T, channels],
     A [channels, N], B, C [T, N]; returns (y [T, channels], S)."""
     S = torch.zeros_like(A) if state is None else state.clone()
     y = torch.zeros_like(x)
